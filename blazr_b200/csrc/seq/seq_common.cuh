@@ -25,6 +25,18 @@ __device__ __forceinline__ void store_act(void* out, int dtype, int64_t idx, flo
     else reinterpret_cast<__nv_bfloat16*>(out)[idx] = __float2bfloat16_rn(v);
 }
 
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store_act4(void* out, int dtype, int64_t idx, const float4 v) {
+    if (dtype == B200SEQ_F32) {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + idx) = v;
+    } else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&lo), u.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + idx) = u;
+    }
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -52,6 +64,23 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return red[32];
 }
 
+// chunk `idx` of a step whose portions are cut into chunks of C tokens from each portion's first token: its entry, first token row and length
+__device__ __forceinline__ bool find_chunk(const b200seq_step& st, int idx, int C, int& e, int& row0, int& len) {
+    int acc = 0;
+    for (e = 0; e < st.B; ++e) {
+        const int s0 = st.ent_start[e], n = st.ent_start[e + 1] - s0;
+        const int nc = (n + C - 1) / C;
+        if (idx < acc + nc) {
+            const int local = idx - acc;
+            row0 = s0 + local * C;
+            len = min(C, n - local * C);
+            return true;
+        }
+        acc += nc;
+    }
+    return false;
+}
+
 __device__ __forceinline__ float sigmoidf_acc(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float siluf_acc(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplusf_acc(float x) { return x > 20.f ? x : log1pf(expf(x)); }
@@ -75,9 +104,11 @@ __device__ __forceinline__ float act_plain(int kind, float z) {
         const float r = fmaxf(z, 0.f);
         return r * r;
     }
+    if (kind == B200SEQ_ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(0.70710678118654752f * z));
+    if (kind == B200SEQ_ACT_TANH) return tanhf(z);
     return z;
 }
 inline bool act_kind_gated(int kind) { return kind == B200SEQ_ACT_SWISH_CLAMP || kind == B200SEQ_ACT_GELU_TANH; }
-inline bool act_kind_known(int kind) { return kind >= B200SEQ_ACT_SWISH_CLAMP && kind <= B200SEQ_ACT_IDENT; }
+inline bool act_kind_known(int kind) { return kind >= B200SEQ_ACT_SWISH_CLAMP && kind <= B200SEQ_ACT_TANH; }
 
 }  // namespace b200seq

@@ -35,7 +35,8 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int64_t l
 }
 
 // choice of one token by one warp: zr = its E router logits; sm = 2 * E + groups floats of shared memory
-// kind 0: sigmoid scores; kind 1: soft-max over the E logits.  corr (or null) is added to the scores for the choice only.
+// kind 0: sigmoid scores; kind 1: soft-max over the E logits; kind 2: choice by the logits, weights = soft-max over the chosen ones.
+// corr (or null) is added to the scores for the choice only.
 __device__ __forceinline__ void route_token(const float* zr, float* sm, int t, int lane, int E, int groups, int keep, int top, int32_t* __restrict__ ids,
                                             float* __restrict__ wts, int32_t* __restrict__ counts, int kind = 0, const float* __restrict__ corr = nullptr) {
     float* s = sm;            // [E] scores
@@ -56,6 +57,11 @@ __device__ __forceinline__ void route_token(const float* zr, float* sm, int t, i
             const float v = s[e] / den;
             s[e] = v, avail[e] = v + (corr ? corr[e] : 0.f);
         }
+    } else if (kind == 2) {
+        float mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zr[e]);
+        mx = warp_max(mx);
+        for (int e = lane; e < E; e += 32) s[e] = expf(zr[e] - mx), avail[e] = zr[e] + (corr ? corr[e] : 0.f);
     } else {
         for (int e = lane; e < E; e += 32) {
             const float v = sigmoidf_acc(zr[e]);
@@ -528,7 +534,7 @@ int b200seq_moe_route(const float* z, int64_t ldz, int T, int E, int groups, int
 
 int b200seq_moe_route_ex(const float* z, int64_t ldz, int T, int E, int groups, int keep, int top, int kind, const float* correction, int32_t* ids, float* wts,
                          int32_t* counts, void* stream) {
-    if (kind != 0 && kind != 1) return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: score kind 0 (sigmoid) or 1 (soft-max)");
+    if (kind < 0 || kind > 2) return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: score kind 0 (sigmoid), 1 (soft-max) or 2 (soft-max over the chosen)");
     if (!z || !ids || !wts || T < 0 || E < 1 || E > MOE_MAX_E || top < 1 || top > E || ldz < E) return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: bad arguments (experts <= %d)", MOE_MAX_E);
     if (groups > 1 && (E % groups || keep < 1 || keep > groups || (int64_t)keep * (E / groups) < top))
         return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: groups must divide the experts and the kept groups must hold `top` experts");
@@ -564,7 +570,7 @@ int b200seq_moe_router(const void* x, int x_dtype, int64_t ldx_, const void* w, 
 
 int b200seq_moe_router_ex(const void* x, int x_dtype, int64_t ldx_, const void* w, int T, int NR, int K, int E, int groups, int keep, int top, int kind,
                           const float* correction, float* z, int64_t ldz, int32_t* ids, float* wts, void* stream) {
-    if (kind != 0 && kind != 1) return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: score kind 0 (sigmoid) or 1 (soft-max)");
+    if (kind < 0 || kind > 2) return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: score kind 0 (sigmoid), 1 (soft-max) or 2 (soft-max over the chosen)");
     if (!x || !w || !z || !ids || !wts || T < 0 || T > 8 || E < 1 || E > MOE_MAX_E || NR < E || K < 1 || ldx_ < K || ldz < NR || top < 1 || top > E)
         return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: bad arguments (at most 8 tokens, experts <= %d)", MOE_MAX_E);
     if (groups > 1 && (E % groups || keep < 1 || keep > groups || (int64_t)keep * (E / groups) < top))

@@ -93,17 +93,6 @@ __global__ void post_norm_kernel(const PostArgs a, const b200seq_step st) {
 // neighbouring elements.  PRE (steps of few rows, bound by latency): every input of the thread's pieces, the norm's weights and the next
 // shift's operands included, is requested before the first is used, so a block pays one round trip to memory instead of one per pass.
 // Without PRE (many rows, bound by bandwidth) only the sum is kept and the small per-column vectors are read where they are used.
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ void store_act4(void* out, int dtype, int64_t idx, const float4 v) {
-    if (dtype == B200SEQ_F32) {
-        *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + idx) = v;
-    } else {
-        __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-        uint2 u;
-        u.x = *reinterpret_cast<uint32_t*>(&lo), u.y = *reinterpret_cast<uint32_t*>(&hi);
-        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + idx) = u;
-    }
-}
 template <int EPT, bool PRE>
 __global__ void post_norm_reg_kernel(const PostArgs a, const b200seq_step st) {
     __shared__ float red[40];

@@ -137,29 +137,13 @@ __global__ void __launch_bounds__(RET_NT) retention_step_kernel(const RetArgs a,
 }
 
 // ---- chunked form -------------------------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ bool ret_find_chunk(const b200seq_step& st, int idx, int& e, int& row0, int& len) {
-    int acc = 0;
-    for (e = 0; e < st.B; ++e) {
-        const int s0 = st.ent_start[e], n = st.ent_start[e + 1] - s0;
-        const int nc = (n + RET_C - 1) / RET_C;
-        if (idx < acc + nc) {
-            const int local = idx - acc;
-            row0 = s0 + local * RET_C;
-            len = min(RET_C, n - local * RET_C);
-            return true;
-        }
-        acc += nc;
-    }
-    return false;
-}
-
 // pass A: grid (V tiles of 64, D tiles of 64, chunks * H).  U[d][v] = sum_i d^(L-1-i) k_i[d] v_i[v]; thread (ty, tx): d = ty * 4 + i, v = tx * 4 + u
 __global__ void __launch_bounds__(RET_NT) retention_local_kernel(const RetArgs a, const b200seq_step st) {
     __shared__ __align__(16) float Ks[RET_C][68];
     __shared__ __align__(16) float Vs[RET_C][68];
     const int c = blockIdx.z / a.H, h = blockIdx.z - c * a.H;
     int e, row0, len;
-    if (!ret_find_chunk(st, c, e, row0, len)) return;
+    if (!find_chunk(st, c, RET_C, e, row0, len)) return;
     const int D = a.D, V = a.V;
     const int v0 = blockIdx.x * 64, d0 = blockIdx.y * 64;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -239,7 +223,7 @@ __global__ void __launch_bounds__(RET_NT) retention_out_kernel(const RetArgs a, 
     __shared__ float pw[RET_C + 1];
     const int c = blockIdx.y, h = blockIdx.z;
     int e, row0, len;
-    if (!ret_find_chunk(st, c, e, row0, len)) return;
+    if (!find_chunk(st, c, RET_C, e, row0, len)) return;
     const int D = a.D, V = a.V, H = a.H;
     const int v0 = blockIdx.x * 64;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;

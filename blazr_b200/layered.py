@@ -1,6 +1,6 @@
 """Layer-list models: a model is a list of layers, each one token mixer (attention over the paged KV pool, or a state-space
 recurrence with per-slot state, retention, or latent attention) plus an optional feed-forward (dense or a mixture of experts),
-wrapped in the pieces a design switches on.  Three layouts of the residual path exist:
+wrapped in the pieces a design switches on.  These layouts of the residual path exist:
   "streams": sublayers in sequence over several residual streams with learned mixing, grouped RMS norms and a short
              carried-state convolution in front of every sublayer (blazr_b200/fenorax.py);
   "depth":   parallel layers (mixer and feed-forward read the same input through two layer norms), one residual stream whose
@@ -11,7 +11,10 @@ wrapped in the pieces a design switches on.  Three layouts of the residual path 
   "out_norm": sublayers in sequence that read the residual itself; the RMS norm sits on the sublayer's OUTPUT, x <- x + norm(sublayer(x));
              a mixer may be two branches side by side (an attention beside an element-wise gated recurrence) whose results are
              summed with fixed scales or after a norm of their own; a hashed bigram table may join the embedding and the logits
-             may pass a soft cap (blazr_b200/pafelorn.py).
+             may pass a soft cap (blazr_b200/pafelorn.py);
+  "sandwich": sublayers in sequence, each normed on both sides, x <- x + norm(sublayer(norm(x))); positions may enter as a sinusoid at the
+             embedding, every layer may add a gated, projected row of a per-token table, and a span of layers may run several times with
+             rows added in front of each pass (blazr_b200/vodelix.py).
 The mechanisms are parameterised (window / chunk / pooled-block size, score scale, unit-norm epsilon, rotary table, gate, state
 size, activation kind, router groups, ...) so that another design can list them in another combination; a design is a function
 config.json -> LayeredConfig.
@@ -101,6 +104,7 @@ class AttentionSpec:
     diff: Optional[float] = None   # differential attention: two maps per head over the same values, o = unit_rms(a1 - lambda a2) * (1 - diff)
     gate_elem: bool = False  # with gated: the sigmoid gate has one logit per output element (heads * vdim) instead of one per head
     kv_from: Optional[int] = None  # the keys and values are those of this (earlier) layer's cache; no k / v tensors of its own
+    unit_sink: bool = False  # one is added to the soft-max denominator (a sink whose logit is 0; no tensor)
 
 
 @dataclass
@@ -161,6 +165,18 @@ class RgLruSpec:
 
 
 @dataclass
+class DeltaSpec:
+    """delta-rule recurrence with a decay and a removal rate per head and key channel: with the unit key u = k / sqrt(sum k^2 + unit_eps),
+    S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T, o_t = S_t^T r; w = exp(-decay_scale sigmoid(W_2 tanh(W_1 h) + w0)), a = sigmoid(W_a h + b);
+    every head's o divided by its root mean square, times a weight and sigmoid(W_g h), then the output projection; f32 state per sequence"""
+    heads: int
+    dim: int                 # per-head key size
+    vdim: int                # per-head value size
+    decay_scale: float
+    unit_eps: float = 1e-6
+
+
+@dataclass
 class TwoBranchSpec:
     """an attention (left) and a recurrence (right) read the same input; result = left_scale * left + right_scale * right, each branch first
     RMS-normed over the model width with a weight of its own when branch_norm"""
@@ -187,7 +203,8 @@ class MoeFfSpec:
     """`top` of `experts` small feed-forwards per token - down(act(up h)), or with a gate branch down(act(gate h, up h)) - plus optionally a
     shared expert of the same form for every token.  router "sigmoid": the choice falls by sigmoid router scores among the experts of the
     `keep` best of `groups` groups of neighbours, weighted by their scores normalised over the chosen, the shared expert times a sigmoid
-    token gate.  router "table": a table indexed by the token id names the experts, each weighted 1 / top, the shared expert is added as it is."""
+    token gate.  router "table": a table indexed by the token id names the experts, each weighted 1 / top, the shared expert is added as it is.
+    router "top_softmax": the largest router logits are chosen and weighted by the soft-max over the chosen ones alone."""
     experts: int
     top: int
     ff: int
@@ -209,10 +226,12 @@ class MoeFfSpec:
 
 @dataclass
 class LayerSpec:
-    kind: str                # "attention" | "ssm" | "retention" | "latent_attention" | "two_branch"
+    kind: str                # "attention" | "ssm" | "retention" | "latent_attention" | "two_branch" | "delta"
     mixer: object
     ff: Optional[object]     # DenseFfSpec | MoeFfSpec | None
-    weights_of: Optional[int] = None   # layout "post": the layer has no tensors of its own and uses those of this (earlier) layer, with its own cache / state
+    weights_of: Optional[int] = None   # layouts "post", "sandwich": the layer has no tensors of its own and uses those of this (earlier) layer, with its own cache / state
+    tensors: Optional[int] = None      # layout "sandwich": the number in the layer's tensor names when it is not its place in the list (layers that run several times)
+    enter: Optional[tuple] = None      # layout "sandwich": added to x in front of this layer: (the embedding output too?, row of "loop.step" or None)
 
 
 @dataclass
@@ -232,6 +251,37 @@ class LayeredConfig:
     post_alpha: float = 1.0      # layout "post": weight of the residual in the sum that is normed
     bigram: Optional[tuple] = None   # layout "out_norm": (buckets, mul_prev, mul_cur) of the hashed bigram table "bigram" [buckets + 1, width]
     logit_softcap: float = 0.0       # > 0: logits <- cap * tanh(logits / cap)
+    norm_shift: float = 0.0          # layout "sandwich": the layer norms' stored weights plus this are what multiplies
+    position_base: float = 0.0       # layout "sandwich": > 0: sin / cos(position * base^(-2i / width)) is added to entries 2i / 2i + 1 of the embedding
+    token_side: int = 0              # layout "sandwich": > 0: every layer adds a row of this size of the table "side.embed", gated and projected
+
+
+class _Rows:
+    """rows of a layer's stacked input projection, with the bias of every row (zero where a projection has none)"""
+
+    def __init__(self, i: int, get, width: int):
+        self.i, self.get, self.w, self.width = i, get, width, 0
+        self.parts, self.biases = [], []
+
+    def add(self, name: str, rows: int, bias: bool = False, perm=None) -> int:
+        """appends tensor `name`; returns its first column in the projection row"""
+        t = self.get(name)
+        if tuple(t.shape) != (rows, self.w):
+            raise ValueError(f"layer {self.i}: {name} has shape {tuple(t.shape)}, expected {(rows, self.w)}")
+        b = self.get(name + ".b").float().reshape(-1) if bias else torch.zeros(rows)
+        if b.numel() != rows:
+            raise ValueError(f"layer {self.i}: {name}.b does not fit")
+        if perm is not None:
+            t, b = perm(t), perm(b)
+        self.parts.append(t.to(torch.bfloat16) if t.dtype != torch.bfloat16 else t)
+        self.biases.append(b)
+        self.width += rows
+        return self.width - rows
+
+    def stacked(self, dev):
+        """(weight bf16 [width, W], bias f32 [width] or None)"""
+        bias = torch.cat(self.biases).to(torch.float32)
+        return torch.cat(self.parts, 0).contiguous().to(dev), (bias.contiguous().to(dev) if bool((bias != 0).any()) else None)
 
 
 class _Workspace:
@@ -275,6 +325,14 @@ class _Workspace:
             self.inner_b = torch.empty((cap, max(1, model.max_rinner)), **act)
             self.conv_a = torch.empty((cap, max(1, model.max_xbc)), **act)
             self.gates = torch.empty((cap, 2 * max(1, model.max_xbc)), **f32)
+            self.ff_inner = torch.empty((cap, max(1, model.max_ff_inner)), **act)
+            self.ff_proj = torch.empty((cap, max(1, model.max_ff_proj)), **f32)
+        if cfg.layout == "sandwich":    # embedding output (looped spans add it again), low-rank decay branch, token-dependent addition, the feed-forward's own buffers
+            self.xbuf = torch.empty((cap, W), **f32)
+            self.low = torch.empty((cap, max(1, model.max_rank)), **act)
+            self.gates = torch.empty((cap, max(1, model.max_wz)), **f32)
+            self.side_z = torch.empty((cap, max(1, cfg.token_side)), **f32)
+            self.side_g = torch.empty((cap, max(1, cfg.token_side)), **act)
             self.ff_inner = torch.empty((cap, max(1, model.max_ff_inner)), **act)
             self.ff_proj = torch.empty((cap, max(1, model.max_ff_proj)), **f32)
         mo = model.moe_dims
@@ -350,14 +408,16 @@ class LayeredModel:
         def hc(pre):    # (in [S], post = out [S] | mix [S, S])
             return vec(pre + "in"), torch.cat([get(pre + "out").float().reshape(-1), get(pre + "mix").float().reshape(-1)]).contiguous().to(dev)
 
-        if cfg.layout not in ("streams", "depth", "post", "out_norm"):
+        if cfg.layout not in ("streams", "depth", "post", "out_norm", "sandwich"):
             raise ValueError(f"unknown residual layout {cfg.layout}")
-        depth, post, outn = cfg.layout == "depth", cfg.layout == "post", cfg.layout == "out_norm"
-        if (depth or post or outn) and (S != 1 or cfg.canon_taps > 1):
-            raise ValueError("the depth-averaged and post-norm layouts have one residual stream and no carried convolution")
+        depth, post, outn, sandwich = (cfg.layout == l for l in ("depth", "post", "out_norm", "sandwich"))
+        if cfg.layout != "streams" and (S != 1 or cfg.canon_taps > 1):
+            raise ValueError("only the layout of several streams has more than one residual stream and carried convolutions")
+        if not sandwich and (cfg.norm_shift or cfg.position_base or cfg.token_side):
+            raise ValueError("shifted norm weights, sinusoidal positions and the token-dependent addition are wired into the sandwich layout")
         self.embed = lin("embed")
         self.head = self.embed if cfg.tied_head else lin("head")
-        self.final_norm = vec("final.norm")
+        self.final_norm = vec("final.norm") + cfg.norm_shift
         self.final_bias = vec("final.norm.b") if post else None
         if tuple(self.embed.shape) != (cfg.vocab, W) or tuple(self.head.shape) != (cfg.vocab, W) or self.final_norm.numel() != W:
             raise ValueError("embedding / head / final norm shapes do not fit the configuration")
@@ -369,6 +429,15 @@ class LayeredModel:
             self.bigram = lin("bigram")
             if tuple(self.bigram.shape) != (int(cfg.bigram[0]) + 1, W) or int(cfg.bigram[0]) < 1:
                 raise ValueError("the bigram table has buckets + 1 rows of the model width")
+        self.pos_freq = seqops.position_frequencies(W, cfg.position_base).to(dev) if cfg.position_base > 0 else None
+        self.side_table = lin("side.embed") if cfg.token_side else None
+        if cfg.token_side and tuple(self.side_table.shape) != (cfg.vocab, cfg.token_side * (1 + max([i if ls.tensors is None else ls.tensors for i, ls in enumerate(cfg.layers)], default=-1))):
+            raise ValueError("the per-token table has one part of the configured size per layer")
+        steps = [ls.enter[1] for ls in cfg.layers if ls.enter is not None and ls.enter[1] is not None]
+        self.loop_step = vec("loop.step") if steps else None
+        if steps and (self.loop_step.dim() != 2 or self.loop_step.shape[0] <= max(steps) or self.loop_step.shape[1] != W):
+            raise ValueError("loop.step has one row of the model width per pass")
+        self.max_rank = self.max_wz = 1      # sandwich layout: low-rank decay branch (its rank, its output width)
         self.layers: List[Dict[str, object]] = []
         self.max_rinner = 1      # out_norm layout: widest recurrent branch
         self.max_proj = self.max_xbc = self.max_inner = 1
@@ -376,13 +445,17 @@ class LayeredModel:
         self.moe_dims = None      # (experts + 1, top, expert ff): largest over the layers
         self.max_q = self.max_qp = self.max_qn = 1      # latent attention: query rows, latent-space query rows, unrotated query parts
         self.max_ctx_r = self.max_ctx_kv = 0            # latent attention: latent size, per-head keys | values of one position
-        self.weight_bytes = self.embed.numel() * 2 + (0 if cfg.tied_head else self.head.numel() * 2) + (self.bigram.numel() * 2 if self.bigram is not None else 0)
+        self.weight_bytes = self.embed.numel() * 2 + (0 if cfg.tied_head else self.head.numel() * 2) + (self.bigram.numel() * 2 if self.bigram is not None else 0) \
+            + (self.side_table.numel() * 2 if self.side_table is not None else 0)
         for i, ls in enumerate(cfg.layers):
             if post:
                 self.layers.append(self._post_layer(i, ls, lin, vec, get))
                 continue
             if outn:
                 self.layers.append(self._out_layer(i, ls, lin, vec, get))
+                continue
+            if sandwich:
+                self.layers.append(self._sandwich_layer(i, ls, lin, vec, get))
                 continue
             L: Dict[str, object] = {"spec": ls}
             p = f"l{i}."
@@ -598,100 +671,26 @@ class LayeredModel:
             att, right, ap = ls.mixer.left, ls.mixer.right, p + "mix.left."
         else:
             raise ValueError(f"layer {i}: mixer kind {ls.kind} is not wired into the out_norm layout")
-        m = att
-        H, G, D, V = m.heads, m.kv_heads, m.dim, m.vdim
-        if H % G or m.values_from_keys or m.pool or m.chunk:
-            raise ValueError(f"layer {i}: attention options that this layout does not wire (or heads not a multiple of kv_heads)")
-        maps = 2 if m.diff is not None else 1
-        shared = m.kv_from is not None
-        if shared:
-            j = m.kv_from
-            src = cfg.layers[j] if 0 <= j < i else None
-            sm = None if src is None else (src.mixer if src.kind == "attention" else src.mixer.left if src.kind == "two_branch" else None)
-            if sm is None or sm.kv_from is not None or (sm.heads, sm.kv_heads, sm.dim, sm.vdim, sm.diff is None) != (H, G, D, V, m.diff is None):
-                raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys of its own and the same head counts and sizes")
-        parts, biases = [], []
-
-        def add(name, rows, bias, perm=None):
-            t = get(name)
-            if tuple(t.shape) != (rows, W):
-                raise ValueError(f"layer {i}: {name} has shape {tuple(t.shape)}, expected {(rows, W)}")
-            b = get(name + ".b").float().reshape(-1) if bias else torch.zeros(rows)
-            if b.numel() != rows:
-                raise ValueError(f"layer {i}: {name}.b does not fit")
-            if perm is not None:
-                t, b = perm(t), perm(b)
-            parts.append(t.to(torch.bfloat16) if t.dtype != torch.bfloat16 else t)
-            biases.append(b)
-
-        # differential attention: the query rows come head by head as [map 1 | map 2]; they are reordered to [key group][map][head of the group] so
-        # that the two maps are 2 H plain query heads over 2 G key heads (query head h' reads key head h' / (H / G)) that share G value heads
-        R = H // G
-        qperm = (lambda t: t.reshape(G, R, 2, D, *t.shape[1:]).transpose(1, 2).reshape(t.shape)) if maps == 2 else None
-        add(ap + "q", H * maps * D, m.bias, qperm)
-        if not shared:
-            add(ap + "k", G * maps * D, m.bias)
-            add(ap + "v", G * V, m.bias)
-        if m.gated:
-            add(ap + "g", H * V if m.gate_elem else H, False)
-        n_att = sum(t.shape[0] for t in parts)
+        rows = _Rows(i, get, W)
+        self._attention_rows(i, att, ap, rows)
+        n_att = rows.width
         rc = {}
         if isinstance(right, MinGruSpec):
             C = right.width
             for nm, b in (("z", True), ("x", True), ("g", False)):
-                rc[nm] = sum(t.shape[0] for t in parts)
-                add(p + "mix.right." + nm, C, b)
+                rc[nm] = rows.width
+                rows.add(p + "mix.right." + nm, C, b)
         elif isinstance(right, RgLruSpec):
             C = right.width
             if right.blocks < 1 or C % right.blocks or not 1 <= right.conv <= 8:
                 raise ValueError(f"layer {i}: blocks must divide the recurrent width, 1..8 convolution taps")
             for nm in ("y", "x"):
-                rc[nm] = sum(t.shape[0] for t in parts)
-                add(p + "mix.right." + nm, C, True)
+                rc[nm] = rows.width
+                rows.add(p + "mix.right." + nm, C, True)
         elif right is not None:
             raise ValueError(f"layer {i}: unknown recurrent branch {type(right).__name__}")
-        L["w_in"] = torch.cat(parts, 0).contiguous().to(dev)
-        bias = torch.cat(biases).to(torch.float32)
-        L["in_bias"] = bias.contiguous().to(dev) if bool((bias != 0).any()) else None
-        L["w_o"] = lin(ap + "o")
-        if tuple(L["w_o"].shape) != (W, H * V):
-            raise ValueError(f"layer {i}: output projection shape does not fit")
-        L["o_bias"] = vec(ap + "o.b") if m.out_bias else None
-        self.weight_bytes += (L["w_in"].numel() + L["w_o"].numel()) * 2
-        rot_freq, rot_scale = None, 1.0
-        if m.rot is not None:
-            if m.rot.dims < 2 or m.rot.dims % 2 or m.rot.dims > D or m.rot.layout not in ("half", "interleaved"):
-                raise ValueError(f"layer {i}: rotary dimensions must be even and at most the head size, layout half or interleaved")
-            fr, rot_scale = m.rot.table()
-            rot_freq = torch.from_numpy(fr).to(dev)
-        L["rot_freq"] = rot_freq
-        if m.qk_norm not in ("none", "head", "full"):
-            raise ValueError(f"layer {i}: unknown q / k norm {m.qk_norm}")
-        L["q_norm_w"] = vec(ap + "q.norm") if m.qk_norm != "none" else None
-        L["k_norm_w"] = vec(ap + "k.norm") if m.qk_norm != "none" and not shared else None
-        nq, nk = (D, D) if m.qk_norm == "head" else (H * maps * D, G * maps * D)
-        if L["q_norm_w"] is not None and (L["q_norm_w"].numel() != nq or (L["k_norm_w"] is not None and L["k_norm_w"].numel() != nk)):
-            raise ValueError(f"layer {i}: q / k norm weights do not fit")
-        if m.qk_norm == "full" and maps == 2:
-            raise ValueError(f"layer {i}: a norm over the whole projection is not wired for differential attention")
-        L["temp"] = vec(ap + "temp") if m.head_temp else None
-        L["sink"] = vec(ap + "sink") if m.sink else None
-        if (L["temp"] is not None and L["temp"].numel() != H) or (L["sink"] is not None and L["sink"].numel() != H) or (maps == 2 and (m.head_temp or m.sink)):
-            raise ValueError(f"layer {i}: one temperature / sink per head (not with differential attention)")
-        L["desc"] = seqops.attn_desc(H * maps, G * maps, D, V, m.scale, gated=m.gated, gate_elem=m.gate_elem, window=m.window,
-                                     qk_eps=cfg.eps if (m.qk_norm != "none" or m.qk_unit_norm) else -1.0, rot_freq=rot_freq, rot_scale=rot_scale, sink=L["sink"],
-                                     q_norm_w=L["q_norm_w"], k_norm_w=L["k_norm_w"], norm_full=m.qk_norm == "full", rot_half=m.rot is not None and m.rot.layout == "half",
-                                     in_bias=L["in_bias"], kv_shared=shared, value_heads=G if maps == 2 else 0, softcap=m.softcap, head_scale=L["temp"],
-                                     keep_first=m.keep_first if m.window > 0 else 0)
-        if L["desc"].width != n_att:
-            raise AssertionError("attention columns of the stacked projection")
-        if maps == 2:
-            for nm in ("lq1", "lk1", "lq2", "lk2"):
-                if get(ap + nm).numel() != D:
-                    raise ValueError(f"layer {i}: {nm} has the head size")
-            f64 = lambda nm: get(ap + nm).to(torch.float64).reshape(-1)
-            L["lambda"] = float(torch.exp((f64("lq1") * f64("lk1")).sum()) - torch.exp((f64("lq2") * f64("lk2")).sum())) + float(m.diff)
-        self.max_inner = max(self.max_inner, H * V * maps)
+        L["w_in"], L["in_bias"] = rows.stacked(dev)
+        self._attention_rest(L, i, att, ap, n_att, lin, vec, get)
         L["rcols"] = rc
         if isinstance(right, MinGruSpec):
             L["w_ro"] = lin(p + "mix.right.o")
@@ -739,10 +738,149 @@ class LayeredModel:
             self.max_ff_inner, self.max_ff_proj = max(self.max_ff_inner, f.ff), max(self.max_ff_proj, f.ff)
         return L
 
-    def _load_moe(self, L, i: int, f: "MoeFfSpec", lin, vec, get) -> None:
+    # ---- attention inside the stacked projection of a layer (layouts "out_norm" and "sandwich") ---------------------------------------------------
+    def _attention_rows(self, i: int, m: "AttentionSpec", ap: str, rows: "_Rows") -> None:
+        """the rows [q | k | v | gate] of an attention"""
+        cfg = self.cfg
+        H, G, D, V = m.heads, m.kv_heads, m.dim, m.vdim
+        if H % G or m.values_from_keys or m.pool or m.chunk:
+            raise ValueError(f"layer {i}: attention options that this layout does not wire (or heads not a multiple of kv_heads)")
+        maps = 2 if m.diff is not None else 1
+        shared = m.kv_from is not None
+        if shared:
+            j = m.kv_from
+            src = cfg.layers[j] if 0 <= j < i else None
+            sm = None if src is None else (src.mixer if src.kind == "attention" else src.mixer.left if src.kind == "two_branch" else None)
+            if sm is None or sm.kv_from is not None or (sm.heads, sm.kv_heads, sm.dim, sm.vdim, sm.diff is None) != (H, G, D, V, m.diff is None):
+                raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys of its own and the same head counts and sizes")
+        # differential attention: the query rows come head by head as [map 1 | map 2]; they are reordered to [key group][map][head of the group] so
+        # that the two maps are 2 H plain query heads over 2 G key heads (query head h' reads key head h' / (H / G)) that share G value heads
+        R = H // G
+        qperm = (lambda t: t.reshape(G, R, 2, D, *t.shape[1:]).transpose(1, 2).reshape(t.shape)) if maps == 2 else None
+        rows.add(ap + "q", H * maps * D, m.bias, qperm)
+        if not shared:
+            rows.add(ap + "k", G * maps * D, m.bias)
+            rows.add(ap + "v", G * V, m.bias)
+        if m.gated:
+            rows.add(ap + "g", H * V if m.gate_elem else H, False)
+
+    def _attention_rest(self, L, i: int, m: "AttentionSpec", ap: str, n_att: int, lin, vec, get) -> None:
+        """output projection, norms, rotation, sinks and the descriptor of an attention whose rows begin the stacked projection L["w_in"]"""
+        cfg, dev, W = self.cfg, self.dev, self.cfg.width
+        H, G, D, V = m.heads, m.kv_heads, m.dim, m.vdim
+        maps, shared = 2 if m.diff is not None else 1, m.kv_from is not None
+        L["w_o"] = lin(ap + "o")
+        if tuple(L["w_o"].shape) != (W, H * V):
+            raise ValueError(f"layer {i}: output projection shape does not fit")
+        L["o_bias"] = vec(ap + "o.b") if m.out_bias else None
+        self.weight_bytes += (L["w_in"].numel() + L["w_o"].numel()) * 2
+        rot_freq, rot_scale = None, 1.0
+        if m.rot is not None:
+            if m.rot.dims < 2 or m.rot.dims % 2 or m.rot.dims > D or m.rot.layout not in ("half", "interleaved"):
+                raise ValueError(f"layer {i}: rotary dimensions must be even and at most the head size, layout half or interleaved")
+            fr, rot_scale = m.rot.table()
+            rot_freq = torch.from_numpy(fr).to(dev)
+        L["rot_freq"] = rot_freq
+        if m.qk_norm not in ("none", "head", "full"):
+            raise ValueError(f"layer {i}: unknown q / k norm {m.qk_norm}")
+        L["q_norm_w"] = vec(ap + "q.norm") if m.qk_norm != "none" else None
+        L["k_norm_w"] = vec(ap + "k.norm") if m.qk_norm != "none" and not shared else None
+        nq, nk = (D, D) if m.qk_norm == "head" else (H * maps * D, G * maps * D)
+        if L["q_norm_w"] is not None and (L["q_norm_w"].numel() != nq or (L["k_norm_w"] is not None and L["k_norm_w"].numel() != nk)):
+            raise ValueError(f"layer {i}: q / k norm weights do not fit")
+        if m.qk_norm == "full" and maps == 2:
+            raise ValueError(f"layer {i}: a norm over the whole projection is not wired for differential attention")
+        L["temp"] = vec(ap + "temp") if m.head_temp else None
+        L["sink"] = vec(ap + "sink") if m.sink else (torch.zeros(H, dtype=torch.float32, device=dev) if m.unit_sink else None)
+        if (L["temp"] is not None and L["temp"].numel() != H) or (L["sink"] is not None and L["sink"].numel() != H) or (maps == 2 and (m.head_temp or m.sink or m.unit_sink)):
+            raise ValueError(f"layer {i}: one temperature / sink per head (not with differential attention)")
+        L["desc"] = seqops.attn_desc(H * maps, G * maps, D, V, m.scale, gated=m.gated, gate_elem=m.gate_elem, window=m.window,
+                                     qk_eps=cfg.eps if (m.qk_norm != "none" or m.qk_unit_norm) else -1.0, rot_freq=rot_freq, rot_scale=rot_scale, sink=L["sink"],
+                                     q_norm_w=L["q_norm_w"], k_norm_w=L["k_norm_w"], norm_full=m.qk_norm == "full", rot_half=m.rot is not None and m.rot.layout == "half",
+                                     in_bias=L["in_bias"], kv_shared=shared, value_heads=G if maps == 2 else 0, softcap=m.softcap, head_scale=L["temp"],
+                                     keep_first=m.keep_first if m.window > 0 else 0)
+        if L["desc"].width != n_att:
+            raise AssertionError("attention columns of the stacked projection")
+        if maps == 2:
+            for nm in ("lq1", "lk1", "lq2", "lk2"):
+                if get(ap + nm).numel() != D:
+                    raise ValueError(f"layer {i}: {nm} has the head size")
+            f64 = lambda nm: get(ap + nm).to(torch.float64).reshape(-1)
+            L["lambda"] = float(torch.exp((f64("lq1") * f64("lk1")).sum()) - torch.exp((f64("lq2") * f64("lk2")).sum())) + float(m.diff)
+        self.max_inner = max(self.max_inner, H * V * maps)
+
+    # ---- layout "sandwich": weights of one layer ----------------------------------------------------------------------------------------------
+    def _sandwich_layer(self, i: int, ls: "LayerSpec", lin, vec, get) -> Dict[str, object]:
+        """a layer that runs again (weights_of) shares every tensor with its first run and gets a cache / state of its own in allocate()"""
+        cfg, dev, W = self.cfg, self.dev, self.cfg.width
+        m, f = ls.mixer, ls.ff
+        n = i if ls.tensors is None else ls.tensors
+        if ls.weights_of is not None:
+            j = ls.weights_of
+            if not 0 <= j < i or cfg.layers[j].weights_of is not None:
+                raise ValueError(f"layer {i}: weights_of must name an earlier layer that has tensors of its own")
+            if cfg.layers[j].kind != ls.kind or cfg.layers[j].mixer != m or cfg.layers[j].ff != f:
+                raise ValueError(f"layer {i}: a layer that shares weights has the sizes of the layer it shares them with")
+            return dict(self.layers[j], spec=ls)
+        L: Dict[str, object] = {"spec": ls}
+        p = f"l{n}."
+
+        def norm(name):
+            w = vec(p + name)
+            if w.numel() != W:
+                raise ValueError(f"layer {i}: {name} does not fit the width")
+            return w
+
+        for q in ("1", "1b") + (("2", "2b") if f is not None else ()):
+            L["norm" + q] = norm("norm" + q) + cfg.norm_shift
+        rows = _Rows(i, get, W)
+        if ls.kind == "attention":
+            if m.diff is not None or m.kv_from is not None or m.out_bias:
+                raise ValueError(f"layer {i}: differential attention, another layer's keys and an output bias are not wired into the sandwich layout")
+            self._attention_rows(i, m, p + "mix.", rows)
+            n_att = rows.width
+            L["w_in"], L["in_bias"] = rows.stacked(dev)
+            self._attention_rest(L, i, m, p + "mix.", n_att, lin, vec, get)
+        elif ls.kind == "delta":
+            H, D, V, ap = m.heads, m.dim, m.vdim, p + "mix."
+            rank = int(get(ap + "w1").shape[0])
+            for nm, r in (("r", H * D), ("k", H * D), ("v", H * V), ("g", H * V), ("a", H * D), ("w1", rank)):
+                rows.add(ap + nm, r)
+            L["w_in"], _ = rows.stacked(dev)
+            L["w_o"], L["w_2"] = lin(ap + "o"), lin(ap + "w2")
+            L["w0"], L["a_b"], L["mnorm"] = vec(ap + "w0"), vec(ap + "a.b"), vec(ap + "norm")
+            if tuple(L["w_o"].shape) != (W, H * V) or tuple(L["w_2"].shape) != (H * D, rank) or L["w0"].numel() != H * D or L["a_b"].numel() != H * D or L["mnorm"].numel() != H * V:
+                raise ValueError(f"layer {i}: delta-rule tensor shapes do not fit the configuration")
+            L["desc"] = seqops.delta_desc(H, D, V, rank, L["w_2"], L["w0"], L["a_b"], L["mnorm"], m.decay_scale, m.unit_eps, cfg.eps)
+            self.max_inner = max(self.max_inner, H * V)
+            self.max_rank, self.max_wz = max(self.max_rank, rank), max(self.max_wz, H * D)
+            self.weight_bytes += (L["w_in"].numel() + L["w_o"].numel() + L["w_2"].numel()) * 2
+        else:
+            raise ValueError(f"layer {i}: mixer kind {ls.kind} is not wired into the sandwich layout")
+        self.max_proj = max(self.max_proj, L["w_in"].shape[0])
+        if isinstance(f, MoeFfSpec):
+            self._load_moe(L, i, f, lin, vec, get, p)
+        elif f is not None:
+            if f.act not in seqops.ACT_KINDS or seqops.ACT_KINDS[f.act] in seqops.ACT_GATED:
+                raise ValueError(f"layer {i}: dense feed-forward activation {f.act} is not a plain kind")
+            L["w_up"], L["w_down"] = lin(p + "mlp.up"), lin(p + "mlp.down")
+            if tuple(L["w_up"].shape) != (f.ff, W) or tuple(L["w_down"].shape) != (W, f.ff):
+                raise ValueError(f"layer {i}: feed-forward tensor shapes do not fit the configuration")
+            self.weight_bytes += (L["w_up"].numel() + L["w_down"].numel()) * 2
+            self.max_ff_inner, self.max_ff_proj = max(self.max_ff_inner, f.ff), max(self.max_ff_proj, f.ff)
+        if cfg.token_side:
+            d = cfg.token_side
+            L["side_gate"], L["side_proj"], L["side_norm"] = lin(p + "side.gate"), lin(p + "side.proj"), norm("side.norm")
+            L["side_col"] = n * d
+            if tuple(L["side_gate"].shape) != (d, W) or tuple(L["side_proj"].shape) != (W, d):
+                raise ValueError(f"layer {i}: shapes of the token-dependent addition do not fit the configuration")
+            self.weight_bytes += (L["side_gate"].numel() + L["side_proj"].numel()) * 2
+        return L
+
+    def _load_moe(self, L, i: int, f: "MoeFfSpec", lin, vec, get, p: Optional[str] = None) -> None:
         """tensors of a mixture-of-experts feed-forward: router (rows of a shared expert's token gate stacked behind it) or table, stacked expert
         weights (gated kinds with alternating gate / up rows), the shared expert"""
-        cfg, W, p = self.cfg, self.cfg.width, f"l{i}."
+        cfg, W, p = self.cfg, self.cfg.width, f"l{i}." if p is None else p
         if f.act not in seqops.ACT_KINDS or not 1 <= f.top <= f.experts + f.identity:
             raise ValueError(f"layer {i}: expert activation {f.act} / top {f.top} is not supported")
         gated = seqops.ACT_KINDS[f.act] in seqops.ACT_GATED
@@ -760,8 +898,8 @@ class LayeredModel:
             if int(t.min()) < 0 or int(t.max()) >= f.experts:
                 raise ValueError(f"layer {i}: the expert table names an expert outside 0..{f.experts - 1}")
             L["table"] = t.to(torch.int32).contiguous().to(self.dev)
-        elif f.router in ("sigmoid", "softmax"):
-            if f.router == "sigmoid" and (f.identity or f.correction):
+        elif f.router in ("sigmoid", "softmax", "top_softmax"):
+            if f.router != "softmax" and (f.identity or f.correction):
                 raise ValueError(f"layer {i}: identity experts and a correction go with the soft-max router")
             router = [p + "mlp.router"] + ([p + "mlp.shared.sg"] if f.shared_ff and f.shared_gate else [])
             L["w_router"] = lin(*router)
@@ -831,6 +969,9 @@ class LayeredModel:
                     L["canon2_state"] = torch.zeros((max_seqs, max(hist, 1), cfg.width), **f32)
             if cfg.layout == "post":
                 L["shift_state"] = torch.zeros((max_seqs, cfg.width), **f32)      # the mixer input of the sequence's last token
+            if ls.kind == "delta":
+                L["delta_state"] = torch.zeros((max_seqs, m.heads, m.dim, m.vdim), **f32)
+                continue
             if cfg.layout == "out_norm":
                 att = m if ls.kind == "attention" else m.left
                 maps = 2 if att.diff is not None else 1
@@ -884,7 +1025,12 @@ class LayeredModel:
                     seen.add(key)
                     need = max([need] + [seqops.attn_scratch_floats(T, 1, key[0], key[1], att.vdim, keys) for T in range(1, cap + 1)])
                 continue
-            if L["spec"].kind == "ssm":
+            if L["spec"].kind == "delta":
+                key = (m.heads, m.dim, m.vdim)
+                if key not in seen:
+                    seen.add(key)
+                    need = max(need, seqops.delta_scratch_floats(cap, self.max_seqs, *key))
+            elif L["spec"].kind == "ssm":
                 need = max(need, seqops.ssm_scratch_floats(cap, self.max_seqs, m.heads, m.vdim, m.state))
             elif L["spec"].kind == "retention":
                 need = max(need, seqops.retention_scratch_floats(cap, self.max_seqs, m.heads, m.dim, m.vdim))
@@ -907,7 +1053,7 @@ class LayeredModel:
         return need
 
     def cache_bytes(self) -> int:
-        keys = ("canon1_state", "canon2_state", "kpool", "vpool", "kpooled", "vpooled", "conv_state", "ssm_state", "shift_state", "ret_state", "rec_state")
+        keys = ("canon1_state", "canon2_state", "kpool", "vpool", "kpooled", "vpooled", "conv_state", "ssm_state", "shift_state", "ret_state", "rec_state", "delta_state")
         return sum(L[k].numel() * 4 for L in self.layers for k in keys if k in L)
 
     def _ctx_buffers(self, rows: int):
@@ -997,6 +1143,8 @@ class LayeredModel:
             self._run_post(ws, T, B, R, debug_layers)
         elif self.cfg.layout == "out_norm":
             self._run_out(ws, T, B, R, debug_layers)
+        elif self.cfg.layout == "sandwich":
+            self._run_sandwich(ws, T, B, R, debug_layers)
         else:
             self._run_streams(ws, T, B, R, sample, debug_layers)
         if R:
@@ -1226,9 +1374,103 @@ class LayeredModel:
         if R and (not n or debug_layers is not None):
             ops.group_rmsnorm(x if R == T and debug_layers is None else x.index_select(0, want.long()), self.final_norm, 1, cfg.eps, ws.fin[:R])
 
+    SIDE_FUSED_ELEMS = 1 << 17      # few tokens: up to this many weights per projection the token-dependent addition runs in one block per token
+
+    def _run_sandwich(self, ws: _Workspace, T: int, B: int, R: int, debug_layers: Optional[list]) -> None:
+        """sublayers in sequence over one residual x (f32), each normed on both sides.  Between sublayers ONE kernel: the norm of the sublayer's
+        result, the residual sum, the rows added in front of a looped span, the next sublayer's norm and its input in the activation type; after
+        the last one the final norm of the wanted rows.  The token-dependent addition reads x as it is; in steps of few tokens it is part of the
+        kernel that closes the sublayer before it."""
+        cfg, ops = self.cfg, seqops
+        st = self._desc(ws, T, B)
+        x, a, y, x0 = ws.h[:T], ws.a[:T], ws.y[:T], ws.xbuf[:T]
+        want, ids = ws.view("want")[:R], ws.view("ids")
+        n = len(self.layers)
+        par = self.overlap_branches and self.dev.type == "cuda" and seqops.timeline is None      # a shared expert beside the routed ones, on a second stream
+        if par and self._side is None:
+            self._side, self._side2 = torch.cuda.Stream(self.dev), torch.cuda.Stream(self.dev)
+
+        def entering(i):
+            e = self.layers[i]["spec"].enter
+            if e is None:
+                return {}
+            return dict(add_row=x0 if e[0] else None, add_vec=self.loop_step[e[1]] if e[1] is not None else None)
+
+        def ending(i):
+            """what the kernel that ends layer i leaves behind: the next layer's input, or the final norm of the wanted rows; with debug_layers x alone"""
+            if debug_layers is not None:
+                return dict(x_out=x)
+            if i + 1 < n:
+                return dict(x_out=x, a_out=a, fin_w=self.layers[i + 1]["norm1"], **entering(i + 1))
+            return dict(a_out=ws.fin[:R], fin_w=self.final_norm, rows=want)
+
+        reads_x0 = any(L["spec"].enter is not None and L["spec"].enter[0] for L in self.layers)
+        first = entering(0) if n else {}
+        ops.embed_pos(self.embed, ids, st, cfg.embed_scale, self.pos_freq, x, cfg.eps, x0=x0 if reads_x0 else None, add_vec=first.get("add_vec"),
+                      fin_w=self.layers[0]["norm1"] if n else None, a=a if n else None)
+        fused_side = T <= 8 and cfg.token_side * cfg.width <= self.SIDE_FUSED_ELEMS
+        for i, L in enumerate(self.layers):
+            ls: LayerSpec = L["spec"]
+            skip = debug_layers is None and i + 1 == n and not R       # nothing wanted: the last layer's results after its mixer are not needed
+            proj = ws.proj[:T, :L["w_in"].shape[0]]
+            ops.linear(a, L["w_in"], proj)
+            if ls.kind == "attention":
+                self._attention_out(L, ls.mixer, ws, st, T, proj, y)
+            else:
+                self._delta(L, ls.mixer, ws, st, T, proj, y)
+            if skip:
+                break
+            open_w = L["norm1b"]       # norm of the result that still has to join the residual
+            if ls.ff is not None:
+                ops.sandwich_norm(x, cfg.eps, y=y, w=open_w, x_out=x, a_out=a, fin_w=L["norm2"])
+                if isinstance(ls.ff, MoeFfSpec):
+                    shared_done = None
+                    if par and ls.ff.shared_ff:
+                        main, fork, shared_done = torch.cuda.current_stream(self.dev), torch.cuda.Event(), torch.cuda.Event()
+                        fork.record(main)
+                        self._side.wait_event(fork)
+                        with torch.cuda.stream(self._side):
+                            self._shared_expert(L, ls.ff, ws, T, a)
+                            shared_done.record(self._side)
+                    self._moe_ff(L, ls.ff, ws, T, a, y, shared_done)
+                else:
+                    mid = ws.ff_inner.view(-1)[:T * ls.ff.ff].view(T, ls.ff.ff)
+                    self._proj_act(ws.ff_proj.view(-1)[:T * ls.ff.ff].view(T, ls.ff.ff), T, a, L["w_up"], ops.ACT_KINDS[ls.ff.act], mid)
+                    ops.linear(mid, L["w_down"], y)
+                open_w = L["norm2b"]
+            if not cfg.token_side:
+                ops.sandwich_norm(x, cfg.eps, y=y, w=open_w, **ending(i))
+            elif fused_side:
+                ops.side_close(x, y, open_w, cfg.eps, L["side_gate"], L["side_proj"], self.side_table, L["side_col"], ids, L["side_norm"], **ending(i))
+            else:
+                ops.sandwich_norm(x, cfg.eps, y=y, w=open_w, x_out=x, a_out=a)
+                z, g = ws.side_z[:T], ws.side_g[:T]
+                ops.linear(a, L["side_gate"], z)
+                ops.token_gate(z, self.side_table, L["side_col"], ids, g)
+                ops.linear(g, L["side_proj"], y)
+                ops.sandwich_norm(x, cfg.eps, y=y, w=L["side_norm"], **ending(i))
+            if debug_layers is not None:
+                debug_layers.append(x.cpu())
+                if i + 1 < n:
+                    ops.sandwich_norm(x, cfg.eps, x_out=x, a_out=a, fin_w=self.layers[i + 1]["norm1"], **entering(i + 1))
+        if R and (not n or debug_layers is not None):
+            ops.sandwich_norm(x, cfg.eps, a_out=ws.fin[:R], fin_w=self.final_norm, rows=want)
+
+    def _delta(self, L, m: DeltaSpec, ws: _Workspace, st, T: int, proj: torch.Tensor, y: torch.Tensor) -> None:
+        H, D, V, d = m.heads, m.dim, m.vdim, L["desc"]
+        o = ws.inner_a.view(-1)[:T * H * V].view(T, H * V)
+        wz = None
+        if st.T != st.B:        # portions: the low-rank branch's second half as one product; single tokens: inside the recurrence's kernel
+            low = ws.low.view(-1)[:T * d.rank].view(T, d.rank)
+            wz = ws.gates.view(-1)[:T * H * D].view(T, H * D)
+            seqops.act(proj[:, d.w_col:d.w_col + d.rank], seqops.ACT_TANH, low)
+            seqops.linear(low, L["w_2"], wz)
+        seqops.delta(proj, st, d, wz, L["delta_state"], o, ws.scratch)
+        seqops.linear(o, L["w_o"], y)
+
     def _attention_out(self, L, m: AttentionSpec, ws: _Workspace, st, T: int, proj: torch.Tensor, y: torch.Tensor) -> None:
-        """attention of the out_norm layout over the layer's own pool or the pool of the layer whose keys and values it shares"""
-        src = L["kv_src"]
+        """attention (prepared from the stacked projection `proj`) over the layer's own pool or the pool of the layer whose keys and values it shares"""
+        src = L.get("kv_src", L)
         seqops.attn_prep_ex(proj, st, L["desc"], L.get("kpool"), L.get("vpool"))
         H, V = m.heads, m.vdim
         o = ws.inner_a.view(-1)[:T * H * V].view(T, H * V)
@@ -1392,13 +1634,14 @@ class LayeredModel:
             pass
         elif f.router == "table":         # no router: the token id names the experts
             ops.moe_table_route(L["table"], ws.view("ids"), T, E, top, ids, wts, None if rows_form else ws.moe_cnt)
-        elif f.router == "softmax":
+        elif f.router in ("softmax", "top_softmax"):
+            kind = ops.ROUTE_SOFTMAX if f.router == "softmax" else ops.ROUTE_TOP_SOFTMAX
             z = ws.moe_z[:T, :L["w_router"].shape[0]]
             if T <= 8 and rows_form:        # few tokens: projection and choice in one kernel
-                ops.moe_router_ex(a, L["w_router"], E, 1, 1, top, ops.ROUTE_SOFTMAX, L["correction"], z, ids, wts)
+                ops.moe_router_ex(a, L["w_router"], E, 1, 1, top, kind, L["correction"], z, ids, wts)
             else:
                 ops.linear(a, L["w_router"], z)
-                ops.moe_route_ex(z, E, 1, 1, top, ops.ROUTE_SOFTMAX, L["correction"], ids, wts, None if rows_form else ws.moe_cnt)
+                ops.moe_route_ex(z, E, 1, 1, top, kind, L["correction"], ids, wts, None if rows_form else ws.moe_cnt)
         else:
             z = ws.moe_z[:T, :L["w_router"].shape[0]]
             if T <= 8 and rows_form:        # few tokens: projection and choice in one kernel

@@ -3,7 +3,7 @@ operators of layer-list models (stream mixing + grouped RMS norm, carried-state 
 over a paged KV pool, the state-space recurrence, gated activations, the depth-averaged residual, mixtures of experts, retention,
 latent attention, per-head projections, token shift + gated post-norm, the branch sum + output norm of two-branch mixers, the bigram
 embedding, PolyNorm, soft caps, differential attention, minGRU and real-gated linear recurrences, soft-max routing with identity experts,
-arg-max).
+the delta rule with per-channel decays, layers normed on both sides with sinusoidal positions and a token-dependent addition, arg-max).
 
 Like blazr_b200/ops.py, PyTorch is plumbing only (device memory, streams); every compute call goes through ctypes.  The library
 is compiled on first use when it is missing (`ensure_built`): a fresh checkout needs nothing but nvcc.  There is no CPU
@@ -27,8 +27,9 @@ LIB_PATH = os.environ.get("B200SEQ_LIB") or os.path.join(_HERE, "lib", "libb200s
 F32, BF16 = 0, 2
 CONV_RESIDUAL, CONV_SILU = 1, 2
 ACT_SWISH_CLAMP, ACT_GELU_TANH, ACT_RELU2, ACT_IDENT = 0, 1, 2, 3   # gated: clamped swish, tanh-gelu gate; plain: squared relu, the product itself
+ACT_GELU_ERF, ACT_TANH = 4, 5                                       # plain: exact gelu, tanh
 ACT_NONE = -1
-ACT_KINDS = {"swish_clamp": ACT_SWISH_CLAMP, "gelu_tanh": ACT_GELU_TANH, "relu2": ACT_RELU2}
+ACT_KINDS = {"swish_clamp": ACT_SWISH_CLAMP, "gelu_tanh": ACT_GELU_TANH, "relu2": ACT_RELU2, "gelu_erf": ACT_GELU_ERF, "tanh": ACT_TANH}
 ACT_GATED = (ACT_SWISH_CLAMP, ACT_GELU_TANH)
 PATH_AUTO, PATH_ROWS, PATH_TILED, PATH_TC = 0, 1, 2, 3
 TC_MIN_ROWS = 32   # b200seq_linear's automatic choice takes the tensor-core path from this many rows
@@ -40,7 +41,8 @@ EXPORTS = ["b200seq_last_error", "b200seq_version", "b200seq_launch_count", "b20
            "b200seq_attn_ex", "b200seq_moe_route", "b200seq_moe_sort", "b200seq_moe_linear", "b200seq_moe_gather", "b200seq_moe_combine", "b200seq_moe_router", "b200seq_moe_table_route", "b200seq_moe_linear_act", "b200seq_head_linear", "b200seq_latent_gather",
            "b200seq_latent_prep", "b200seq_rotary", "b200seq_retention", "b200seq_retention_scratch_floats", "b200seq_token_shift", "b200seq_post_norm",
            "b200seq_moe_route_ex", "b200seq_moe_router_ex", "b200seq_moe_combine_ex", "b200seq_causal_conv_ex", "b200seq_embed_bigram", "b200seq_branch_norm", "b200seq_polynorm", "b200seq_softcap",
-           "b200seq_diff_combine", "b200seq_min_gru", "b200seq_rg_lru"]
+           "b200seq_diff_combine", "b200seq_min_gru", "b200seq_rg_lru", "b200seq_delta", "b200seq_delta_scratch_floats", "b200seq_embed_pos", "b200seq_sandwich_norm",
+           "b200seq_token_gate", "b200seq_side_close"]
 
 
 class SeqError(RuntimeError):
@@ -79,6 +81,24 @@ def retention_desc(H: int, D: int, V: int, decay: torch.Tensor, eps: float, k_sc
     d = RetentionDesc(H, D, V, 0, H * D, 2 * H * D, 2 * H * D + H * V, decay.data_ptr(), eps, 2 * rot_freq.numel() if rot_freq is not None else 0, int(rot_half),
                       rot_freq.data_ptr() if rot_freq is not None else None, rot_scale, k_scale)
     d.width = 2 * H * D + 2 * H * V
+    return d
+
+
+class DeltaDesc(C.Structure):
+    """b200seq_delta_desc: sizes, columns of the projection row, weights and constants of one delta-rule layer"""
+    _fields_ = [("H", C.c_int32), ("D", C.c_int32), ("V", C.c_int32), ("r_col", C.c_int32), ("k_col", C.c_int32), ("v_col", C.c_int32), ("g_col", C.c_int32),
+                ("a_col", C.c_int32), ("w_col", C.c_int32), ("rank", C.c_int32), ("w2", C.c_void_p), ("w0", C.c_void_p), ("a_b", C.c_void_p), ("norm_w", C.c_void_p),
+                ("decay_scale", C.c_float), ("unit_eps", C.c_float), ("eps", C.c_float)]
+
+
+def delta_desc(H: int, D: int, V: int, rank: int, w2: torch.Tensor, w0: torch.Tensor, a_b: torch.Tensor, norm_w: torch.Tensor, decay_scale: float, unit_eps: float,
+               eps: float) -> "DeltaDesc":
+    """descriptor for a projection row laid out r | k | v | gate | removal logits | low rank; w2 bf16 [H * D, rank], the vectors f32; the caller keeps the tensors alive"""
+    assert w2.dtype == torch.bfloat16 and w2.is_contiguous() and tuple(w2.shape) == (H * D, rank)
+    assert all(t.dtype == torch.float32 and t.numel() == n for t, n in ((w0, H * D), (a_b, H * D), (norm_w, H * V)))
+    cols = [0, H * D, 2 * H * D, 2 * H * D + H * V, 2 * H * (D + V), 3 * H * D + 2 * H * V]
+    d = DeltaDesc(H, D, V, *cols, rank, w2.data_ptr(), w0.data_ptr(), a_b.data_ptr(), norm_w.data_ptr(), decay_scale, unit_eps, eps)
+    d.width = cols[-1] + rank
     return d
 
 
@@ -526,13 +546,13 @@ def argmax(logits: torch.Tensor, ids: torch.Tensor):
 
 
 # ---- layers with the norm on the sublayer's output, two-branch mixers, gated linear recurrences ----------------------------------------------
-ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_TOP_SOFTMAX = 0, 1, 2
 
 
 @_timed
 def moe_route_ex(z: torch.Tensor, E: int, groups: int, keep: int, top: int, kind: int, correction: Optional[torch.Tensor], ids: torch.Tensor, wts: torch.Tensor,
                  counts: Optional[torch.Tensor]):
-    """moe_route with the score kind (ROUTE_SIGMOID / ROUTE_SOFTMAX over the E logits) and a correction f32 [E] that enters the choice only"""
+    """moe_route with the score kind (ROUTE_SIGMOID / ROUTE_SOFTMAX over the E logits / ROUTE_TOP_SOFTMAX over the chosen ones) and a correction f32 [E] that enters the choice only"""
     T, _, ldz = _rows2d(z)
     assert ids.dtype == torch.int32 and wts.dtype == torch.float32 and ids.is_contiguous() and wts.is_contiguous() and ids.numel() >= T * top
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
@@ -633,3 +653,72 @@ def rg_lru(u: torch.Tensor, gates: torch.Tensor, gate_bias: Optional[torch.Tenso
     assert out.is_contiguous() and out.shape[1] == Cn and state.is_contiguous() and state.shape[1] == Cn and sp_lam.numel() == Cn
     _check(lib().b200seq_rg_lru(_p(u), C.c_int64(ldu), _p(gates), C.c_int64(ldg), _p(gate_bias), _p(sp_lam), C.c_float(decay_c), _p(proj), C.c_int64(ldp), y_col, _p(bias),
                                 _p(state), C.byref(step), Cn, blocks, _p(out), _DT[out.dtype], _st(proj)))
+
+
+# ---- delta rule; layers normed on both sides of every sublayer ---------------------------------------------------------------------------------
+def delta_scratch_floats(T: int, B: int, H: int, D: int, V: int) -> int:
+    """floats of work area a delta-rule step of T tokens in B entries wants (0: every entry brings one token)"""
+    f = lib().b200seq_delta_scratch_floats
+    f.restype = C.c_size_t
+    return int(f(T, B, H, D, V))
+
+
+@_timed
+def delta(proj: torch.Tensor, step: "StepDesc", d: "DeltaDesc", wz: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor, scratch: Optional[torch.Tensor] = None):
+    """wz f32 [T, H * D]: low-rank branch output (steps with portions; None in steps of single tokens, where the kernel applies w2 itself)"""
+    _, _, ld = _rows2d(proj)
+    assert out.is_contiguous() and state.is_contiguous() and (scratch is None or (scratch.dtype == torch.float32 and scratch.is_contiguous()))
+    _check(lib().b200seq_delta(_p(proj), C.c_int64(ld), C.byref(step), C.byref(d), _p(wz), C.c_int64(wz.stride(0) if wz is not None else 0), _p(state), _p(out),
+                               _DT[out.dtype], _p(scratch), C.c_size_t(scratch.numel() if scratch is not None else 0), _st(proj)))
+
+
+def position_frequencies(width: int, base: float) -> torch.Tensor:
+    """f32 [2, ceil(width / 2)]: base^(-2i / width) as high and low parts"""
+    import numpy as np
+    f = base ** (-2.0 * np.arange((width + 1) // 2, dtype=np.float64) / width)
+    hi = f.astype(np.float32)
+    return torch.from_numpy(np.stack([hi, (f - hi.astype(np.float64)).astype(np.float32)]))
+
+
+@_timed
+def embed_pos(table: torch.Tensor, ids: torch.Tensor, step: "StepDesc", scale: float, freq: Optional[torch.Tensor], x: torch.Tensor, eps: float, *,
+              x0: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None, fin_w: Optional[torch.Tensor] = None, a: Optional[torch.Tensor] = None):
+    """x[t] = table[ids[t]] * scale + sinusoid(pos) (+ add_vec); x0: the same without add_vec; a: x, normed with fin_w when given, in its own type"""
+    W = x.shape[-1]
+    assert table.dtype == torch.bfloat16 and table.is_contiguous() and x.is_contiguous() and (freq is None or tuple(freq.shape) == (2, (W + 1) // 2))
+    _check(lib().b200seq_embed_pos(_p(table), _p(ids), C.byref(step), C.c_float(scale), _p(freq), W, _p(x0), _p(add_vec), _p(x), _p(fin_w), C.c_float(eps), _p(a),
+                                   _DT[a.dtype] if a is not None else F32, _st(x)))
+
+
+@_timed
+def sandwich_norm(x: torch.Tensor, eps: float, *, y: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, add_row: Optional[torch.Tensor] = None,
+                  add_vec: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, x_out: Optional[torch.Tensor] = None, a_out: Optional[torch.Tensor] = None,
+                  fin_w: Optional[torch.Tensor] = None):
+    """n = x + rms_norm(y) * w + add_row + add_vec; x_out = n, a_out = n (normed with fin_w when given); rows: only these token rows (a_out is row-compact)"""
+    W = x.shape[-1]
+    R = x.shape[0] if rows is None else rows.numel()
+    assert x.is_contiguous() and (y is None or y.is_contiguous()) and (a_out is None or a_out.is_contiguous()) and (add_row is None or add_row.is_contiguous())
+    _check(lib().b200seq_sandwich_norm(_p(x), _p(y), _p(w), C.c_float(eps), _p(add_row), _p(add_vec), W, _p(rows), R, _p(x_out), _p(a_out),
+                                       _DT[a_out.dtype] if a_out is not None else F32, _p(fin_w), _st(x)))
+
+
+@_timed
+def token_gate(z: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor, out: torch.Tensor):
+    """out[t] = gelu_tanh(z[t]) * table[ids[t]][col : col + dim]"""
+    T, dim, ldz = _rows2d(z)
+    assert table.dtype == torch.bfloat16 and table.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, dim)
+    _check(lib().b200seq_token_gate(_p(z), C.c_int64(ldz), T, dim, _p(table), C.c_int64(table.shape[1]), col, _p(ids), _p(out), _DT[out.dtype], _st(z)))
+
+
+@_timed
+def side_close(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, gate: torch.Tensor, proj: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor,
+               side_w: torch.Tensor, *, add_row: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, x_out: Optional[torch.Tensor] = None,
+               a_out: Optional[torch.Tensor] = None, fin_w: Optional[torch.Tensor] = None):
+    """sandwich_norm of a sublayer's result, the token-dependent addition and the next norm in one kernel (steps of few tokens; a block per row)"""
+    W = x.shape[1]
+    R = x.shape[0] if rows is None else rows.numel()
+    dim = gate.shape[0]
+    assert x.is_contiguous() and y.is_contiguous() and tuple(gate.shape) == (dim, W) and tuple(proj.shape) == (W, dim) and gate.is_contiguous() and proj.is_contiguous()
+    assert gate.dtype == proj.dtype == table.dtype == torch.bfloat16 and table.is_contiguous()
+    _check(lib().b200seq_side_close(_p(x), _p(y), _p(w), C.c_float(eps), _p(gate), _p(proj), _p(table), C.c_int64(table.shape[1]), col, dim, _p(ids), _p(side_w),
+                                    _p(add_row), _p(add_vec), W, _p(rows), R, _p(x_out), _p(a_out), _DT[a_out.dtype] if a_out is not None else F32, _p(fin_w), _st(x)))

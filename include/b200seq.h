@@ -8,7 +8,8 @@
  * post-norm residual, the residual with the norm on the sublayer's output and two-branch mixers, weighted
  * q / k norms, soft-capped scores, kept first positions, differential attention, minGRU and real-gated
  * linear recurrences, PolyNorm, soft-max routing with identity experts, a hashed bigram embedding,
- * arg-max sampling.
+ * the delta rule with per-channel decays, layers normed on both sides with sinusoidal positions and a
+ * token-dependent addition, arg-max sampling.
  *
  * It sits beside libb200q (include/b200q.h), which holds the quantized linear layer; the conventions are
  * the same:
@@ -145,6 +146,8 @@ int b200seq_ssm_scan(const float* proj, int64_t ldp, int z0, int dt0, const floa
 #define B200SEQ_ACT_GELU_TANH 1
 #define B200SEQ_ACT_RELU2 2
 #define B200SEQ_ACT_IDENT 3 /* plain kind: the product itself, written in out_dtype (a projection whose result feeds the next linear layer) */
+#define B200SEQ_ACT_GELU_ERF 4 /* plain kind: 0.5 z (1 + erf(z / sqrt(2))) */
+#define B200SEQ_ACT_TANH 5     /* plain kind: tanh(z) */
 
 /* out = act(x . w^T), the product itself never reaches memory.  w: bf16 [N, K]; out [M, N / 2] (gated kinds) or [M, N] (plain kinds) in
  * out_dtype, row stride ldo.  M <= 8: weight-streaming rows (f32 or bf16 activations); more rows: the tensor-core path, which needs bf16
@@ -319,7 +322,8 @@ int b200seq_moe_combine(const float* ys, const float* wts, const int32_t* slot_o
                         float* y, void* stream);
 
 /* ---- the same choice with soft-max scores and a correction -------------------------------------------------------------------------------
- * kind 0: s = sigmoid(z) (b200seq_moe_route); kind 1: s = softmax(z[0 .. E)) in f32.  correction (f32 [E] or null) is added to s for the
+ * kind 0: s = sigmoid(z) (b200seq_moe_route); kind 1: s = softmax(z[0 .. E)) in f32; kind 2: the choice falls by the logits themselves and the
+ * weights are the soft-max over the chosen logits only (s = exp(z - max z), normalised over the chosen).  correction (f32 [E] or null) is added to s for the
  * CHOICE only; the weights are the chosen s / (their sum + 1e-20).  E counts every router output, identity experts included. */
 int b200seq_moe_route_ex(const float* z, int64_t ldz, int T, int E, int groups, int keep, int top, int kind, const float* correction, int32_t* ids, float* wts,
                          int32_t* counts, void* stream);
@@ -375,6 +379,47 @@ int b200seq_min_gru(const float* proj, int64_t ldp, int z_col, int x_col, int g_
                     int out_dtype, void* stream);
 int b200seq_rg_lru(const float* u, int64_t ldu, const float* gates, int64_t ldg, const float* gate_bias, const float* sp_lam, float decay_c, const float* proj,
                    int64_t ldp, int y_col, const float* bias, float* state, const b200seq_step* st, int C, int blocks, void* out, int out_dtype, void* stream);
+
+/* ---- delta rule with a decay per key channel --------------------------------------------------------------------------------------------------
+ * Columns of the f32 projection row: r at r_col (H*D), k at k_col (H*D), v at v_col (H*V), gate at g_col (H*V), removal logits at a_col (H*D),
+ * the low-rank branch's first half at w_col (rank).  Per head, with state[slot][H][D][V] (f32, read as zero when ent_pos0 == 0):
+ *   u = k / sqrt(sum k^2 + unit_eps);  w = exp(-decay_scale * sigmoid(z + w0)), z = w2 . tanh(row[w_col ..]);  a = sigmoid(row[a_col ..] + a_b)
+ *   S_t = diag(w) S_(t-1) - (a * u) (u^T S_(t-1)) + k v^T   (both products read the old state);   o_t = S_t^T r
+ *   out[t][h] = o_t / sqrt(mean(o_t^2) + eps) * norm_w[h] * sigmoid(gate_t[h])      (act dtype [T, H*V])
+ * Steps in which every entry brings one token run one kernel that applies w2 (bf16 [H*D][rank]) itself; other steps read z from wz (f32 [T, H*D],
+ * row stride ldw), cut the portions into chunks that run in parallel and need b200seq_delta_scratch_floats(...) floats (16-byte aligned).
+ * decay_scale: at most 1.875 (products of one chunk's decays stay in range); D <= 256 in steps with portions. */
+typedef struct b200seq_delta_desc {
+    int32_t H, D, V;
+    int32_t r_col, k_col, v_col, g_col, a_col, w_col, rank;
+    const void* w2;
+    const float *w0, *a_b, *norm_w;
+    float decay_scale, unit_eps, eps;
+} b200seq_delta_desc;
+size_t b200seq_delta_scratch_floats(int T, int B, int H, int D, int V);
+int b200seq_delta(const float* proj, int64_t ld, const b200seq_step* st, const b200seq_delta_desc* d, const float* wz, int64_t ldw, float* state, void* out,
+                  int out_dtype, float* scratch, size_t scratch_floats, void* stream);
+
+/* ---- residual path of layers normed on both sides of every sublayer ---------------------------------------------------------------------------
+ * embed_pos: e[t] = table[ids[t]] * scale + sinusoid, entry 2i = sin(pos * f_i), entry 2i + 1 = cos(pos * f_i); freq: device f32 [2][(W + 1) / 2],
+ * the f_i as high and low parts (f_i = high + low), or null (no positions).  x0[t] <- e (optional), x[t] <- e + add_vec (add_vec [W] optional),
+ * a[t] <- fin_w ? rms_norm(x[t], eps) * fin_w : x[t] in a_dtype (a optional).
+ * sandwich_norm, one block per row r (token t = rows ? rows[r] : r):
+ *   n = x[t] + (y ? rms_norm(y[t], eps) * w : 0) + add_row[t] + add_vec     (add_row f32 [T, W], add_vec f32 [W]: each optional)
+ *   x_out[t] <- n (optional, may be x);   a_out[r] <- fin_w ? rms_norm(n, eps) * fin_w : n, in out_dtype (optional) */
+int b200seq_embed_pos(const void* table_bf16, const int32_t* ids, const b200seq_step* st, float scale, const float* freq, int W, float* x0, const float* add_vec, float* x,
+                      const float* fin_w, float eps, void* a, int a_dtype, void* stream);
+int b200seq_sandwich_norm(const float* x, const float* y, const float* w, float eps, const float* add_row, const float* add_vec, int W, const int32_t* rows, int R,
+                          float* x_out, void* a_out, int out_dtype, const float* fin_w, void* stream);
+/* An addition that depends on the token id: g[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][col + j] (table bf16, row stride ldt; z f32, g in out_dtype
+ * [T, dim]); its projection back to the model width is normed and added by sandwich_norm.
+ * side_close: the whole of it for steps of few tokens, a block per row as in sandwich_norm: n1 = x + rms_norm(y) * w;  z = gate . n1 (bf16 [dim, W]);  g as above;
+ * n = n1 + rms_norm(proj . g) * side_w + add_row + add_vec (proj bf16 [W, dim]);  outputs as sandwich_norm. */
+int b200seq_token_gate(const float* z, int64_t ldz, int T, int dim, const void* table_bf16, int64_t ldt, int col, const int32_t* ids, void* out, int out_dtype,
+                       void* stream);
+int b200seq_side_close(const float* x, const float* y, const float* w, float eps, const void* gate_bf16, const void* proj_bf16, const void* table_bf16, int64_t ldt, int col,
+                       int dim, const int32_t* ids, const float* side_w, const float* add_row, const float* add_vec, int W, const int32_t* rows, int R,
+                       float* x_out, void* a_out, int out_dtype, const float* fin_w, void* stream);
 
 /* ids[r] = argmax_v logits[r][v] (first maximum) */
 int b200seq_argmax(const float* logits, int R, int V, int32_t* ids, void* stream);
