@@ -92,7 +92,9 @@ struct ActParams {
     float limit, alpha, shift;
 };
 __device__ __forceinline__ bool act_is_gated(int kind) { return kind == B200SEQ_ACT_SWISH_CLAMP || kind == B200SEQ_ACT_GELU_TANH; }
-__device__ __forceinline__ float gelu_tanhf_acc(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// 0.5 (1 + tanh(u)) as sigmoid(2 u), and 0.5 (1 + erf(u)) as 0.5 erfc(-u): no cancellation for negative arguments, where the result may be normed next
+__device__ __forceinline__ float gelu_tanhf_acc(float z) { return z * sigmoidf_acc(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
+__device__ __forceinline__ float gelu_erff_acc(float z) { return 0.5f * z * erfcf(-0.70710678118654752f * z); }
 __device__ __forceinline__ float act_gated(const ActParams& a, float gate, float up) {
     if (a.kind == B200SEQ_ACT_GELU_TANH) return gelu_tanhf_acc(gate) * up;
     const float g = fminf(gate, a.limit);
@@ -104,7 +106,7 @@ __device__ __forceinline__ float act_plain(int kind, float z) {
         const float r = fmaxf(z, 0.f);
         return r * r;
     }
-    if (kind == B200SEQ_ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(0.70710678118654752f * z));
+    if (kind == B200SEQ_ACT_GELU_ERF) return gelu_erff_acc(z);
     if (kind == B200SEQ_ACT_TANH) return tanhf(z);
     return z;
 }

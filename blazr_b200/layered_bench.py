@@ -6,12 +6,14 @@ dense-attention decoder (blazr_b200/decode.py, Q8_0 weights) of the same width, 
     kernels  : every operator of one prefill step and one decode step timed alone (CUDA events around each launch), with its
                algorithmic bytes / FLOPs and the fraction of the roofline it reaches; the like kernels of the decoder beside them
 
-`python bench.py --layered fenorax|gemosun|teselix|pafelorn [--layered-sizes w1024,w2048]` prints the result as one JSON line; bench.py's default
+`python bench.py --layered fenorax|gemosun|teselix|pafelorn|vodelix [--layered-sizes w1024,w2048]` prints the result as one JSON line; bench.py's default
 workload and JSON line are untouched.  For Gemosun (parallel attention / feed-forward layers, three of four feed-forwards a mixture of
 experts) the closest existing model, Fenorax at the same sizes, runs beside it as well; for Teselix (retention and latent-attention mixers,
 table-routed experts) both run beside it: Gemosun is the closest in attention and experts, Fenorax in the recurrence.  For Pafelorn (windowed
 attention beside element-wise recurrences, differential attention, soft-max-routed gated experts) Gemosun (windowed attention with rotation,
-routed experts) and Fenorax (a recurrence with carried state and a short convolution) run beside it as well.
+routed experts) and Fenorax (a recurrence with carried state and a short convolution) run beside it as well.  For Vodelix (a delta rule with a
+matrix state per head, unmasked causal attention, routed plain experts) Teselix (retention: a matrix state per head; experts) and Gemosun (plain
+experts behind a learned router) run beside it as well.
 """
 from __future__ import annotations
 
@@ -94,6 +96,55 @@ def pafelorn_config(sz: dict, experts: int = 32, identity: int = 2, top: int = 4
                        {"type": "parallel", "mixer": {"left": left1, "right": {"width": W}, "left_scale": 1.0, "right_scale": 1.0}, "mlp": moe},
                        {"type": "parallel_2", "mixer": {"left": left2, "right": {"width": W, "blocks": 8, "conv": 4}}, "mlp": dict(dense)},
                        {"type": "attention", "mixer": dict(diff, kv_from=0), "mlp": dict(moe)}]}
+
+
+def vodelix_config(sz: dict, experts: int = 32, top: int = 4) -> dict:
+    """four runs of three sandwich-norm layers [delta rule + dense, attention + experts (twice), delta rule + experts] of the size's width and head
+    layout; an expert is a quarter of the dense size; the token-dependent addition has a sixteenth of the width"""
+    H, D, W = sz["heads"], sz["dim"], sz["width"]
+    eff = sz["ff"] // 4
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top}, "shared": {"ff": eff}}
+    delta = {"type": "general_delta", "mixer": {"heads": H, "dim": D}}
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": sz["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5}}
+    return {"architecture": "Vodelix", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "token_side": {"dim": W // 16}, "loop": {"start": 1, "stop": 2, "times": 2},
+            "layers": [dict(delta, mlp={"kind": "dense", "ff": sz["ff"]}), dict(att, mlp=moe), dict(delta, mlp=dict(moe))]}
+
+
+def random_tensors_vodelix(cfg: dict, device, seed: int = 7, rank: int = 64):
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W, V, n, sd = cfg["width"], cfg["vocab"], len(cfg["layers"]), cfg["token_side"]["dim"]
+
+    def rnd(*shape, scale=1.0):
+        return (torch.randn(shape, generator=g, device=device) * scale).to(torch.bfloat16)
+
+    zeros, ones = (lambda *s: torch.zeros(*s, dtype=torch.bfloat16, device=device)), (lambda *s: torch.ones(*s, dtype=torch.bfloat16, device=device))
+    t = {"embed": rnd(V, W), "final.norm": zeros(W), "loop.step": rnd(cfg["loop"]["times"], W, scale=0.1), "side.embed": rnd(V, n * sd)}
+    lin = lambda name, o, i: t.__setitem__(name, rnd(o, i, scale=i ** -0.5))
+    for i, lay in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", lay["mixer"], lay["mlp"]
+        for nm in ("norm1", "norm1b", "norm2", "norm2b"):
+            t[p + nm] = zeros(W)
+        H, D = m["heads"], m["dim"]
+        if lay["type"] == "attention":
+            G, Vd = m["kv_heads"], m["vdim"]
+            lin(p + "mix.q", H * D, W), lin(p + "mix.k", G * D, W), lin(p + "mix.v", G * Vd, W), lin(p + "mix.o", W, H * Vd)
+            t[p + "mix.q.norm"], t[p + "mix.k.norm"] = ones(H * D), ones(G * D)
+        else:
+            for nm in "rkvga":
+                lin(p + "mix." + nm, H * D, W)
+            lin(p + "mix.w1", rank, W), lin(p + "mix.w2", H * D, rank), lin(p + "mix.o", W, H * D)
+            t[p + "mix.w0"], t[p + "mix.a.b"], t[p + "mix.norm"] = rnd(H * D) - 3.0, zeros(H * D), ones(H * D)
+        if f["kind"] == "dense":
+            lin(p + "mlp.up", f["ff"], W), lin(p + "mlp.down", W, f["ff"])
+        else:
+            lin(p + "mlp.router", f["router"]["experts"], W)
+            for e in range(f["router"]["experts"]):
+                lin(p + f"mlp.e{e}.up", f["expert"]["ff"], W), lin(p + f"mlp.e{e}.down", W, f["expert"]["ff"])
+            lin(p + "mlp.shared.up", f["shared"]["ff"], W), lin(p + "mlp.shared.down", W, f["shared"]["ff"])
+        lin(p + "side.gate", sd, W), lin(p + "side.proj", W, sd)
+        t[p + "side.norm"] = ones(W)
+    return lambda name: t[name].cpu()
 
 
 def random_tensors_pafelorn(cfg: dict, device, seed: int = 7):
@@ -271,10 +322,23 @@ def _events():
 
 def _linear_weights(model: LayeredModel) -> int:
     """weights of the linear layers a token goes through (of a mixture of experts: the router, the chosen experts, the shared one)"""
-    n = sum(L[k].numel() for L in model.layers for k in ("w_in", "w_o", "w_gu", "w_down", "w_router", "w_sup", "w_sdown", "rg1", "rg2", "w_uq", "w_ukT", "w_uv", "w_up", "w_ro", "w_gates") if k in L)
+    n = sum(L[k].numel() for L in model.layers for k in ("w_in", "w_o", "w_gu", "w_down", "w_router", "w_sup", "w_sdown", "rg1", "rg2", "w_uq", "w_ukT", "w_uv", "w_up", "w_ro", "w_gates", "w_2", "side_gate", "side_proj") if k in L)
     for L in model.layers:
         if "w_eup" in L:
             n += L["spec"].ff.top * (L["w_eup"][0].numel() + L["w_edown"][0].numel())
+    return n
+
+
+def _touched_bytes(model: LayeredModel, B: int) -> int:
+    """weight bytes a step of B single tokens streams: all weights but the experts no token of the step chose (at most B * top of a layer's experts
+    are touched) and the per-token table; layers that run several times count every time"""
+    n = model.weight_bytes - (model.side_table.numel() * 2 if model.side_table is not None else 0)
+    for L in model.layers:
+        if L["spec"].weights_of is not None and model.cfg.layout == "sandwich":
+            n += 2 * sum(v.numel() for k, v in L.items() if isinstance(v, torch.Tensor) and v.dtype == torch.bfloat16)
+        if "w_eup" in L:
+            E_, per = L["w_eup"].shape[0], (L["w_eup"][0].numel() + L["w_edown"][0].numel()) * 2
+            n -= (E_ - min(E_, B * L["spec"].ff.top)) * per
     return n
 
 
@@ -316,6 +380,29 @@ def _cost(name: str, shapes, scal, scen: dict, kw: dict = None):
         if scen["prefill"]:
             flops += 2.0 * T * d.H * 32 * (d.D + d.V)                                       # on average 32 of the chunk's 64 keys are at or before a token
         return T * (ld * 4 + d.H * d.V * sh[2][1]) + 2 * B * d.H * d.D * d.V * 4, flops, "f32" if scen["prefill"] else "hbm"
+    if name == "delta":           # the projection row (and the low-rank branch's rows) in, the gated result out, the state of every entry read and written
+        d = scen["delta_desc"]
+        T, ld = sh[0][0]
+        wz = T * d.H * d.D * 4 if scen["prefill"] else d.H * d.D * d.rank * 2
+        # u^T S, decay, removal, k v^T, S^T r of the plain recurrence (the chunked form's own products are not counted)
+        return T * (ld * 4 + d.H * d.V * kw.get("out_es", 2)) + wz + 2 * scen["entries"] * d.H * d.D * d.V * 4, 9.0 * T * d.H * d.D * d.V, "f32" if scen["prefill"] else "hbm"
+    if name == "sandwich_norm":   # x, the result and the added rows in; x and / or the activation rows out
+        rows = kw["rows"][0][0] if isinstance(kw.get("rows"), tuple) else sh[0][0][0]
+        W = sh[0][0][1]
+        reads = 1 + sum(1 for n in ("y", "add_row") if isinstance(kw.get(n), tuple))
+        outs = sum(kw[n][1] for n in ("x_out", "a_out") if isinstance(kw.get(n), tuple))
+        return rows * W * (4 * reads + outs), 0.0, "hbm"
+    if name == "side_close":      # x and the result in, both projections once, x and the activation rows out
+        rows = kw["rows"][0][0] if isinstance(kw.get("rows"), tuple) else sh[0][0][0]
+        W = sh[0][0][1]
+        outs = sum(kw[n][1] for n in ("x_out", "a_out") if isinstance(kw.get(n), tuple))
+        return rows * W * (8 + outs) + by(sh[3]) + by(sh[4]), 0.0, "hbm"
+    if name == "token_gate":      # logits and table rows in, gated rows out
+        (T, dim) = sh[0][0]
+        return T * dim * (4 + 2 + sh[-1][1]), 0.0, "hbm"
+    if name == "embed_pos":       # table rows in; x, the embedding output and the activation rows out
+        (T, W) = sh[-1][0]
+        return T * W * (2 + 4 + sum(kw[n][1] for n in ("x0", "a") if isinstance(kw.get(n), tuple))), 0.0, "hbm"
     if name == "latent_gather":   # pool rows in, latents out in the activation type
         (rows, R), es = sh[-1][0], sh[-1][1]
         return rows * R * (4 + es), 0.0, "hbm"
@@ -436,19 +523,23 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
     elif design.lower() == "pafelorn":
         cfg = pafelorn_config(sz)
         model = LayeredModel(registry.LAYERED["Pafelorn"](cfg), random_tensors_pafelorn(cfg, dev), dev, dtype)
+    elif design.lower() == "vodelix":
+        cfg = vodelix_config(sz)
+        model = LayeredModel(registry.LAYERED["Vodelix"](cfg), random_tensors_vodelix(cfg, dev, rank={1024: 64, 2048: 96}.get(sz["width"], 128)), dev, dtype)
     else:
         raise ValueError(f"no synthetic workload for design '{design}'")
-    gem, tes, paf = design.lower() == "gemosun", design.lower() == "teselix", design.lower() == "pafelorn"
+    gem, tes, paf, vod = (design.lower() == n for n in ("gemosun", "teselix", "pafelorn", "vodelix"))
     pool = 16 if gem else 0
     desc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.AttnDesc)), None)
     rdesc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.RetentionDesc)), None)
+    ddesc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.DeltaDesc)), None)
     Bmax = max(batches)
     eng = Engine(model, max_tokens=max(S, Bmax * (ctx + steps + 64)) + 64, max_seqs=Bmax, max_step_tokens=max(S, 2048), prefill_chunk=S)
     rng = np.random.default_rng(3)
     prompt = rng.integers(0, sz["vocab"], S).tolist()
     out = {"size": size, "config": {k: sz[k] for k in sz}, "layers": [l["type"] + ("+" + l["mlp"].get("kind", "ff") if l["mlp"] else "") for l in cfg["layers"]],
            "streams": cfg.get("streams", 1), "linear_weights": _linear_weights(model), "weight_bytes": model.weight_bytes}
-    if gem or tes or paf:
+    if gem or tes or paf or vod:
         r = cfg["layers"][1]["mlp"]
         out["experts"] = {"experts": r["router"]["experts"], "top": r["router"]["top"], "ff": r["expert"]["ff"], "shared_ff": r["shared"]["ff"], "groups": r["router"].get("groups")}
     lin_flops_tok = 2.0 * (_linear_weights(model) + 0)
@@ -483,6 +574,8 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
     if gem:     # window of `chunk` positions plus one pooled entry per block of 16 wholly before it
         vis = np.minimum(pos + 1, chunk) + np.maximum(0, (pos - chunk + 1) // pool)
         scen = dict(prefill=True, entries=1, visible_keys=int(vis.sum()), kv_rows_touched=S + S // pool, attn_desc=desc0)
+    elif vod:   # every earlier position
+        scen = dict(prefill=True, entries=1, visible_keys=int((pos + 1).sum()), kv_rows_touched=S, attn_desc=desc0, delta_desc=ddesc0)
     elif paf:   # a sliding window of `chunk` positions (the few kept first positions of one layer are not counted)
         scen = dict(prefill=True, entries=1, visible_keys=int(np.minimum(pos + 1, chunk).sum()), kv_rows_touched=S, attn_desc=desc0)
     elif tes:   # every earlier position; a step of portions attends over per-head keys projected from the gathered latents
@@ -522,19 +615,14 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
         e1.record()
         torch.cuda.synchronize()
         msd_e2e = e0.elapsed_time(e1) / steps
-        # weights a step streams: all of them but the experts no token of the step chose (at most B * top of a layer's experts are touched)
-        touched = model.weight_bytes
-        for L in model.layers:
-            if "w_eup" in L:
-                E_, per = L["w_eup"].shape[0], (L["w_eup"][0].numel() + L["w_edown"][0].numel()) * 2
-                touched -= (E_ - min(E_, B * L["spec"].ff.top)) * per
+        touched = _touched_bytes(model, B)
         row = {"batch": B, "context": ctx, "ms_per_step": round(msd, 4), "tokens_per_s": round(B / msd * 1e3, 1), "e2e_tokens_per_s": round(B / msd_e2e * 1e3, 1),
                "weight_bytes_touched": touched, "weight_GBs": round(touched / (msd * 1e-3) / 1e9, 1),
                "frac_hbm_weights_only": round(touched / (msd * 1e-3) / 1e9 / pk["hbm_gbs"], 3)}
         held = eng.cache.live[ids[0]].n_tokens
         lo = (held // chunk) * chunk
-        seen = (min(held + 1, chunk) + max(0, (held - chunk + 1) // pool)) if gem else (held + 1 if tes else (min(held + 1, chunk) if paf else held - lo + 1))
-        scen = dict(prefill=False, entries=B, visible_keys=B * seen, kv_rows_touched=B * seen, attn_desc=desc0, ret_desc=rdesc0)
+        seen = (min(held + 1, chunk) + max(0, (held - chunk + 1) // pool)) if gem else (held + 1 if tes or vod else (min(held + 1, chunk) if paf else held - lo + 1))
+        scen = dict(prefill=False, entries=B, visible_keys=B * seen, kv_rows_touched=B * seen, attn_desc=desc0, ret_desc=rdesc0, delta_desc=ddesc0)
         row["kernels"] = kernel_table(model, eng, dec_step, scen, pk)
         out["decode"].append(row)
         for r in ids:
@@ -690,7 +778,7 @@ def run(design: str, sizes: List[str], pk, pk_kind: str, S: int = 4096, ctx: int
     for size in sizes:
         row = {"size": size}
         row[design.lower()] = bench_layered(design, size, pk, S=S, ctx=ctx, steps=steps)
-        others = {"fenorax": [], "gemosun": ["fenorax"], "teselix": ["gemosun", "fenorax"], "pafelorn": ["gemosun", "fenorax"]}.get(design.lower(), ["fenorax"])
+        others = {"fenorax": [], "gemosun": ["fenorax"], "teselix": ["gemosun", "fenorax"], "pafelorn": ["gemosun", "fenorax"], "vodelix": ["teselix", "gemosun"]}.get(design.lower(), ["fenorax"])
         for other in others:                # the closest existing layer-list models at the same sizes
             try:
                 row[other] = bench_layered(other, size, pk, S=S, ctx=ctx, steps=steps)

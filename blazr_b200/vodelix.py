@@ -80,7 +80,7 @@ def _feed_forward(mlp, where: str):
     if kind == "moe":
         r, ex, shared = _need(mlp, "router", where), _need(mlp, "expert", where), mlp.get("shared")
         spec = MoeFfSpec(experts=_size(r, "experts", where + ".router"), top=_size(r, "top", where + ".router"), ff=_size(ex, "ff", where + ".expert"), act=EXPERT_ACT,
-                         router="top_softmax", shared_ff=_size(shared, "ff", where + ".shared") if shared else 0, shared_gate=False)
+                         router="top_softmax", shared_ff=_size(shared, "ff", where + ".shared") if shared is not None else 0, shared_gate=False)
         if spec.top > spec.experts:
             raise ConfigError(f"config: {where}: router.top must lie between 1 and router.experts")
         return spec
@@ -104,7 +104,7 @@ def parse_config(cfg: dict) -> LayeredConfig:
     side = cfg.get("token_side")
     out = LayeredConfig(name=ARCHITECTURE, vocab=_size(cfg, "vocab", "top level"), width=_size(cfg, "width", "top level"), streams=1, norm_groups=1,
                         eps=float(_need(_need(cfg, "norm", "top level"), "eps", "norm")), canon_taps=0, embed_scale=1.0, layout="sandwich", tied_head=True,
-                        depth_average=False, norm_shift=1.0, position_base=POSITION_BASE, token_side=_size(side, "dim", "token_side") if side else 0)
+                        depth_average=False, norm_shift=1.0, position_base=POSITION_BASE, token_side=_size(side, "dim", "token_side") if side is not None else 0)
     layers = []
     for i, lay in enumerate(_need(cfg, "layers", "top level")):
         where = f"layers[{i}]"

@@ -180,8 +180,8 @@ def forward(cfg: dict, P: Dict[str, torch.Tensor], tokens: List[int], layers_out
 
 
 # ---- random checkpoints ------------------------------------------------------------------------------------------------------------
-def random_model(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
-    """random weights that are exact in bfloat16 (so that float32 runs of the framework see the same numbers)"""
+def random_model(cfg: dict, seed: int = 0, rank: int = 7) -> Dict[str, torch.Tensor]:
+    """random weights that are exact in bfloat16 (so that float32 runs of the framework see the same numbers); rank: size of the low-rank decay branch"""
     gen = torch.Generator().manual_seed(seed)
     W, Vc, n = cfg["width"], cfg["vocab"], len(cfg["layers"])
     P: Dict[str, torch.Tensor] = {}
@@ -210,7 +210,6 @@ def random_model(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             lin(q + "q", H * D, W), lin(q + "k", G * D, W), lin(q + "v", G * V, W), lin(q + "o", W, H * V)
             P[q + "q.norm"], P[q + "k.norm"] = rnd(H * D, std=0.3, mean=1.0), rnd(G * D, std=0.3, mean=1.0)
         else:
-            rank = m.get("_rank", 7)      # the low-rank branch's size is the tensors' alone
             for nm in "rkvga":
                 lin(q + nm, H * D, W, gain=1.5 if nm == "k" else 1.0)
             P[q + "a.b"], P[q + "w0"], P[q + "norm"] = rnd(H * D, std=0.5), rnd(H * D, std=1.0, mean=-1.5), rnd(H * D, std=0.3, mean=1.0)
@@ -224,7 +223,7 @@ def random_model(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             if f.get("shared"):
                 lin(p + "mlp.shared.up", f["shared"]["ff"], W, gain=2.0), lin(p + "mlp.shared.down", W, f["shared"]["ff"])
         if sd:
-            lin(p + "side.gate", sd, W, gain=1.5), lin(p + "side.proj", W, sd)
+            lin(p + "side.gate", sd, W, gain=0.3), lin(p + "side.proj", W, sd)      # (logits far below zero everywhere would leave the norm behind it nothing but rounding)
             P[p + "side.norm"] = rnd(W, std=0.2, mean=0.6)
     return P
 
