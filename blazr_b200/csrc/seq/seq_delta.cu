@@ -24,9 +24,9 @@ namespace b200seq {
 
 constexpr int DL_C = 32;     // tokens per chunk
 constexpr int DL_NT = 256;
-constexpr int DL_AS = DL_C + 4;   // row stride of the score matrices
-constexpr int DL_VT = 16;    // value columns per block of pass B
-constexpr int DL_SS = 18;    // row stride of pass B's state tile
+constexpr int DL_AS = DL_C + 4;       // row stride of a 32 x 32 matrix
+constexpr int DL_MS = 2 * DL_C + 4;   // row stride of two of them side by side
+constexpr int DL_VS = 68;             // row stride of a tile of 64 value columns
 
 struct DeltaArgs {
     const float* proj;
@@ -44,17 +44,19 @@ struct DeltaArgs {
     int out_dtype;
 };
 
-// record of one (chunk, head): P' [C][Dp] | beta W_C [C][Dp] | R' [C][Dp] | W_C [Dp] | U, then the start state [Dp][Vp] | O0 [C][Vp]
+// record of one (chunk, head): P' [C][Ds] | beta W_C [C][Ds] | W_C [Dp] | R' [C][Ds] | U, then the start state [Dp][Vp] | O0 [C][Vp].  Rows of key
+// channels keep the row stride they have in shared memory, so that a block copies them as they lie.
+__host__ __device__ constexpr int delta_up4(int n) { return (n + 3) & ~3; }
+__host__ __device__ constexpr int delta_ds(int D) { return delta_up4(D) + 4; }
 struct DeltaRec {
-    int Dp, Vp;
-    __host__ __device__ DeltaRec(int D, int V) : Dp((D + 3) & ~3), Vp((V + 3) & ~3) {}
-    __host__ __device__ int64_t p() const { return 0; }
-    __host__ __device__ int64_t b() const { return (int64_t)DL_C * Dp; }
-    __host__ __device__ int64_t r() const { return (int64_t)2 * DL_C * Dp; }
-    __host__ __device__ int64_t w() const { return (int64_t)3 * DL_C * Dp; }
-    __host__ __device__ int64_t u() const { return w() + Dp; }
-    __host__ __device__ int64_t o() const { return u() + (int64_t)Dp * Vp; }
-    __host__ __device__ int64_t size() const { return o() + (int64_t)DL_C * Vp; }
+    int Ds, Dp, Vp;
+    __host__ __device__ constexpr DeltaRec(int D, int V) : Ds(delta_ds(D)), Dp(delta_up4(D)), Vp(delta_up4(V)) {}
+    __host__ __device__ constexpr int b() const { return DL_C * Ds; }
+    __host__ __device__ constexpr int w() const { return 2 * DL_C * Ds; }
+    __host__ __device__ constexpr int r() const { return w() + Dp; }
+    __host__ __device__ constexpr int u() const { return r() + DL_C * Ds; }
+    __host__ __device__ constexpr int o() const { return u() + Dp * Vp; }
+    __host__ __device__ constexpr int size() const { return o() + DL_C * Vp; }
 };
 
 __device__ __forceinline__ float delta_decay(float z, float scale) { return expf(-scale * sigmoidf_acc(z)); }
@@ -166,30 +168,47 @@ __global__ void __launch_bounds__(DL_NT) delta_step_kernel(const DeltaArgs a, co
     }
 }
 
+// The passes are compiled for D = V = TD (64, 128) and in a general form (TD = 0).
 // ---- pass A: grid (chunks, H) -----------------------------------------------------------------------------------------------------------
-// Dynamic shared memory: P | R | B | K [C][Ds] (B and K next to each other: one operand of 2 C rows; P and R likewise) | four transposed score
-// matrices [C (j)][AS] | decays [C][Ds] in the same place as V and Y tiles 2 x [C][68] | products of the decays per segment [4][Dp] | W_C [Dp]
-__host__ __device__ inline int delta_ds(int D) { return ((D + 3) & ~3) + 4; }
-__host__ __device__ inline int delta_local_floats(int D) {
-    const int Ds = delta_ds(D), Dp = (D + 3) & ~3;
-    const int wd = DL_C * Ds, vy = 2 * DL_C * 68;
-    return 4 * DL_C * Ds + 4 * DL_C * DL_AS + (wd > vy ? wd : vy) + 5 * Dp;
+// Dynamic shared memory: P | R | B | K [C][Ds] (P and R, B and K next to each other: operands of 2 C rows) | T: L transposed, then (I + L)^-1
+// transposed [C][AS] | F transposed [C][AS] | M | E transposed [C][MS] | decays [C][Ds] in the same place as V and Y tiles 2 x [C][VS] |
+// products of the decays per segment [4][Dp] | W_C [Dp]
+__host__ __device__ constexpr int delta_local_floats(int D) {
+    const int wd = DL_C * delta_ds(D), vy = 2 * DL_C * DL_VS;
+    return 4 * DL_C * delta_ds(D) + 2 * DL_C * DL_AS + DL_C * DL_MS + (wd > vy ? wd : vy) + 5 * delta_up4(D);
 }
 
-__global__ void __launch_bounds__(DL_NT, 2) delta_local_kernel(const DeltaArgs a, const b200seq_step st) {
+// acc[8][4] += A^T[0 .. kn)[8 rows] * B[0 .. kn)[4 columns]
+template <int SIGN>
+__device__ __forceinline__ void delta_mm84(float (&acc)[8][4], const float* A, int as, const float* B, int bs, int kn) {
+#pragma unroll 4
+    for (int k = 0; k < kn; ++k) {
+        const float4 a0 = ld4(A + k * as), a1 = ld4(A + k * as + 4), b = ld4(B + k * bs);
+        const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float x = SIGN > 0 ? av[i] : -av[i];
+            acc[i][0] = fmaf(x, b.x, acc[i][0]), acc[i][1] = fmaf(x, b.y, acc[i][1]), acc[i][2] = fmaf(x, b.z, acc[i][2]), acc[i][3] = fmaf(x, b.w, acc[i][3]);
+        }
+    }
+}
+
+template <int TD>
+__global__ void __launch_bounds__(DL_NT, TD == 64 ? 3 : (TD == 128 ? 2 : 1)) delta_local_kernel(const DeltaArgs a, const b200seq_step st) {
     extern __shared__ __align__(16) float sm[];
-    const int D = a.D, V = a.V, H = a.H, Ds = delta_ds(D), Dp = (D + 3) & ~3;
+    const int D = TD ? TD : a.D, V = TD ? TD : a.V, H = a.H;
+    const DeltaRec rec(D, V);
+    const int Ds = rec.Ds, Dp = rec.Dp, Vp = rec.Vp;
     float *P = sm, *R = P + DL_C * Ds, *B = R + DL_C * Ds, *K = B + DL_C * Ds;
-    float *AL = K + DL_C * Ds, *AM = AL + DL_C * DL_AS, *AF = AM + DL_C * DL_AS, *AE = AF + DL_C * DL_AS;
-    float* Wd = AE + DL_C * DL_AS;
-    float *Vs = Wd, *Ys = Wd + DL_C * 68;
-    const int wd = DL_C * Ds, vy = 2 * DL_C * 68;
+    float *AT = K + DL_C * Ds, *AF = AT + DL_C * DL_AS, *ME = AF + DL_C * DL_AS;
+    float* Wd = ME + DL_C * DL_MS;
+    float *Vs = Wd, *Ys = Wd + DL_C * DL_VS;
+    const int wd = DL_C * Ds, vy = 2 * DL_C * DL_VS;
     float* segp = Wd + (wd > vy ? wd : vy);
     float* wc = segp + 4 * Dp;
     const int c = blockIdx.x, h = blockIdx.y;
     int e, row0, len;
     if (!find_chunk(st, c, DL_C, e, row0, len)) return;
-    const DeltaRec rec(D, V);
     float* out = a.chunk + ((int64_t)c * H + h) * rec.size();
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
     // the tokens' rows: a warp takes four tokens
@@ -199,7 +218,9 @@ __global__ void __launch_bounds__(DL_NT, 2) delta_local_kernel(const DeltaArgs a
         const bool in = i < len;
         const float* row = a.proj + (int64_t)(row0 + i) * a.ld;
         float ss = 0.f;
-        for (int d = lane; d < Dp; d += 32) {
+#pragma unroll
+        for (int d0 = 0; d0 < Dp; d0 += 32) {
+            const int d = d0 + lane;
             float k = 0.f, r = 0.f, av = 0.f, w = 1.f;
             if (in && d < D) {
                 const int cc = h * D + d;
@@ -208,10 +229,13 @@ __global__ void __launch_bounds__(DL_NT, 2) delta_local_kernel(const DeltaArgs a
                 w = delta_decay(a.wz[(int64_t)(row0 + i) * a.ldw + cc] + a.w0[cc], a.decay_scale);
             }
             ss = fmaf(k, k, ss);
-            K[i * Ds + d] = k, R[i * Ds + d] = r, B[i * Ds + d] = av, Wd[i * Ds + d] = w;
+            if (d < Dp) K[i * Ds + d] = k, R[i * Ds + d] = r, B[i * Ds + d] = av, Wd[i * Ds + d] = w;
         }
         const float uinv = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
-        for (int d = lane; d < Dp; d += 32) {
+#pragma unroll
+        for (int d0 = 0; d0 < Dp; d0 += 32) {
+            const int d = d0 + lane;
+            if (d >= Dp) break;
             const float u = K[i * Ds + d] * uinv;
             P[i * Ds + d] = u, B[i * Ds + d] *= u;
         }
@@ -252,12 +276,13 @@ __global__ void __launch_bounds__(DL_NT, 2) delta_local_kernel(const DeltaArgs a
         for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+#pragma unroll 2
         for (int d = 0; d < Dp; d += 4) {
             float4 q[4], k[4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) q[i] = *reinterpret_cast<const float4*>(P + (ty * 4 + i) * Ds + d);
+            for (int i = 0; i < 4; ++i) q[i] = ld4(P + (ty * 4 + i) * Ds + d);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) k[j] = *reinterpret_cast<const float4*>(B + (tx + 16 * j) * Ds + d);
+            for (int j = 0; j < 4; ++j) k[j] = ld4(B + (tx + 16 * j) * Ds + d);
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -273,186 +298,214 @@ __global__ void __launch_bounds__(DL_NT, 2) delta_local_kernel(const DeltaArgs a
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int cj = tx + 16 * (j & 1);
-                float* m = isp ? (j < 2 ? AL : AM) : (j < 2 ? AF : AE);
-                m[cj * DL_AS + ri] = (isp ? cj < ri : cj <= ri) ? s[i][j] : 0.f;
+                const float v = (isp ? cj < ri : cj <= ri) ? s[i][j] : 0.f;
+                if (j < 2) (isp ? AT : AF)[cj * DL_AS + ri] = v;
+                else ME[cj * DL_MS + (isp ? 0 : DL_C) + ri] = v;
             }
         }
     }
     __syncthreads();
-    // value tiles of 64 columns: Y0 and O0 (one column per thread), then U
+    const int rg = wid & 3;            // products of 32 rows: a warp takes eight rows, a lane four columns; rows before the group's last one enter only
+    const int kn = 8 * (rg + 1);
     for (int v0 = 0; v0 < V; v0 += 64) {
-        __syncthreads();   // the decays (first tile) or the previous tile are done with
-        for (int it = tid; it < DL_C * 64; it += DL_NT) {
+        for (int it = tid; it < DL_C * 64; it += DL_NT) {      // (the scores' barrier, or the end of the previous tile, freed the place)
             const int i = it >> 6, cc = it & 63;
-            Vs[i * 68 + cc] = (i < len && v0 + cc < V) ? a.proj[(int64_t)(row0 + i) * a.ld + a.v_col + (int64_t)h * V + v0 + cc] : 0.f;
+            Vs[i * DL_VS + cc] = (i < len && v0 + cc < V) ? a.proj[(int64_t)(row0 + i) * a.ld + a.v_col + (int64_t)h * V + v0 + cc] : 0.f;
         }
         __syncthreads();
-        if (v0 == 0 && tid < Dp) {   // P' and R', one column (key channel) per thread (D <= the block's threads)
-            const int d = tid;
-            float x[DL_C], r[DL_C];
-    #pragma unroll
-            for (int i = 0; i < DL_C; ++i) x[i] = P[i * Ds + d], r[i] = R[i * Ds + d];
-    #pragma unroll
+        const int nc = (v0 == 0 ? Dp : 0) + 64;                // columns of [P | M V]: P with the first tile only
+        const int pc = v0 == 0 ? Dp : 0;
+        if (wid >= 4) {                                        // M V to the Y tile, E V to the record: 64 rows, the warp's lanes cover 16 column groups of two row groups
+            const int t2 = tid - 128, cg = t2 & 15, rr = t2 >> 4;
+            float acc[8][4];
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) acc[i][u] = 0.f;
+            delta_mm84<1>(acc, ME + rr * 8, DL_MS, Vs + cg * 4, DL_VS, DL_C);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float4 v = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+                if (rr < 4) *reinterpret_cast<float4*>(Ys + (rr * 8 + i) * DL_VS + cg * 4) = v;
+                else if (v0 + cg * 4 < Vp) *reinterpret_cast<float4*>(out + rec.o() + ((rr - 4) * 8 + i) * Vp + v0 + cg * 4) = v;
+            }
+        } else if (wid == 0 && v0 == 0) {                      // (I + L)^-1: lane = column, forward substitution
+            float x[DL_C];
+#pragma unroll
+            for (int i = 0; i < DL_C; ++i) x[i] = i == lane ? 1.f : 0.f;
+#pragma unroll
             for (int j = 0; j < DL_C; ++j) {
                 const float y = x[j];
-    #pragma unroll
+#pragma unroll
                 for (int i4 = j & ~3; i4 < DL_C; i4 += 4) {
-                    const float4 l = *reinterpret_cast<const float4*>(AL + j * DL_AS + i4), f = *reinterpret_cast<const float4*>(AF + j * DL_AS + i4);
+                    const float4 l = ld4(AT + j * DL_AS + i4);
                     x[i4] = fmaf(-l.x, y, x[i4]), x[i4 + 1] = fmaf(-l.y, y, x[i4 + 1]), x[i4 + 2] = fmaf(-l.z, y, x[i4 + 2]), x[i4 + 3] = fmaf(-l.w, y, x[i4 + 3]);
-                    r[i4] = fmaf(-f.x, y, r[i4]), r[i4 + 1] = fmaf(-f.y, y, r[i4 + 1]), r[i4 + 2] = fmaf(-f.z, y, r[i4 + 2]), r[i4 + 3] = fmaf(-f.w, y, r[i4 + 3]);
                 }
             }
-    #pragma unroll
-            for (int i = 0; i < DL_C; ++i) {
-                out[rec.p() + (int64_t)i * Dp + d] = x[i];
-                out[rec.r() + (int64_t)i * Dp + d] = r[i];
+            __syncwarp();
+#pragma unroll
+            for (int i4 = 0; i4 < DL_C; i4 += 4) *reinterpret_cast<float4*>(AT + lane * DL_AS + i4) = make_float4(x[i4], x[i4 + 1], x[i4 + 2], x[i4 + 3]);
+        } else if (v0 == 0) {                                  // beta W_C to the record
+            for (int it = tid - 32; it < DL_C * (Dp >> 2); it += 96) {
+                const int i = it / (Dp >> 2), d = 4 * (it - i * (Dp >> 2));
+                const float4 b = ld4(B + i * Ds + d), w = ld4(wc + d);
+                *reinterpret_cast<float4*>(out + rec.b() + i * Ds + d) = make_float4(b.x * w.x, b.y * w.y, b.z * w.z, b.w * w.w);
             }
-        }
-        // Y0 and O0, one value column per thread: the block's last two warps, beside the P' columns of its first ones
-        if (tid >= DL_NT - 64) {
-            const int cc = tid - (DL_NT - 64);
-            float x[DL_C], o[DL_C];
-#pragma unroll
-            for (int i = 0; i < DL_C; ++i) x[i] = 0.f, o[i] = 0.f;
-#pragma unroll
-            for (int j = 0; j < DL_C; ++j) {
-                const float y = x[j], vv = Vs[j * 68 + cc];
-#pragma unroll
-                for (int i4 = j & ~3; i4 < DL_C; i4 += 4) {
-                    const float4 l = *reinterpret_cast<const float4*>(AL + j * DL_AS + i4), m = *reinterpret_cast<const float4*>(AM + j * DL_AS + i4);
-                    const float4 f = *reinterpret_cast<const float4*>(AF + j * DL_AS + i4), g = *reinterpret_cast<const float4*>(AE + j * DL_AS + i4);
-                    x[i4] = fmaf(m.x, vv, fmaf(-l.x, y, x[i4])), x[i4 + 1] = fmaf(m.y, vv, fmaf(-l.y, y, x[i4 + 1]));
-                    x[i4 + 2] = fmaf(m.z, vv, fmaf(-l.z, y, x[i4 + 2])), x[i4 + 3] = fmaf(m.w, vv, fmaf(-l.w, y, x[i4 + 3]));
-                    o[i4] = fmaf(g.x, vv, fmaf(-f.x, y, o[i4])), o[i4 + 1] = fmaf(g.y, vv, fmaf(-f.y, y, o[i4 + 1]));
-                    o[i4 + 2] = fmaf(g.z, vv, fmaf(-f.z, y, o[i4 + 2])), o[i4 + 3] = fmaf(g.w, vv, fmaf(-f.w, y, o[i4 + 3]));
-                }
-            }
-            const bool in = v0 + cc < rec.Vp;
-#pragma unroll
-            for (int i = 0; i < DL_C; ++i) {
-                Ys[i * 68 + cc] = x[i];
-                if (in) out[rec.o() + (int64_t)i * rec.Vp + v0 + cc] = o[i];
-            }
-        }
-        for (int it = v0 == 0 ? tid : DL_C * Dp; it < DL_C * Dp; it += DL_NT) {
-            const int i = it / Dp, d = it - i * Dp;
-            out[rec.b() + it] = B[i * Ds + d] * wc[d];
         }
         __syncthreads();
+        // [P' | Y0] = (I + L)^-1 [P | M V], in place: column groups dealt to the two halves of the block, results held back until every warp has read
+        constexpr int NG = TD ? (TD + 64 + 255) / 256 : 2;     // column groups a lane may have (D <= 256)
+        float acc[NG][8][4];
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+            const int col = 4 * (lane + 32 * ((wid >> 2) + 2 * g));
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) acc[g][i][u] = 0.f;
+            if (col < pc) delta_mm84<1>(acc[g], AT + rg * 8, DL_AS, P + col, Ds, kn);
+            else if (col < nc) delta_mm84<1>(acc[g], AT + rg * 8, DL_AS, Ys + col - pc, DL_VS, kn);
+        }
+        __syncthreads();
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+            const int col = 4 * (lane + 32 * ((wid >> 2) + 2 * g));
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float4 v = make_float4(acc[g][i][0], acc[g][i][1], acc[g][i][2], acc[g][i][3]);
+                const int r = rg * 8 + i;
+                if (col < pc) {
+                    *reinterpret_cast<float4*>(P + r * Ds + col) = v;
+                    *reinterpret_cast<float4*>(out + r * Ds + col) = v;
+                } else if (col < nc) {
+                    *reinterpret_cast<float4*>(Ys + r * DL_VS + col - pc) = v;
+                }
+            }
+        }
+        __syncthreads();
+        // R' = rho - F P', O0 = E V - F Y0
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+            const int col = 4 * (lane + 32 * ((wid >> 2) + 2 * g));
+            const bool isp = col < pc;
+            if (col >= nc || (!isp && v0 + col - pc >= Vp)) continue;
+            float* dst = isp ? out + rec.r() + rg * 8 * Ds + col : out + rec.o() + rg * 8 * Vp + v0 + col - pc;
+            const int ds = isp ? Ds : Vp;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float4 v = isp ? ld4(R + (rg * 8 + i) * Ds + col) : ld4(dst + i * Vp);
+                acc[g][i][0] = v.x, acc[g][i][1] = v.y, acc[g][i][2] = v.z, acc[g][i][3] = v.w;
+            }
+            if (isp) delta_mm84<-1>(acc[g], AF + rg * 8, DL_AS, P + col, Ds, kn);
+            else delta_mm84<-1>(acc[g], AF + rg * 8, DL_AS, Ys + col - pc, DL_VS, kn);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) *reinterpret_cast<float4*>(dst + i * ds) = make_float4(acc[g][i][0], acc[g][i][1], acc[g][i][2], acc[g][i][3]);
+        }
+        // U = W_C (kappa^T V - beta^T Y0): thread (ty, tx): channels ty * 4 + i, value columns tx * 4 + u
         const int tx = tid & 15, ty = tid >> 4;
+#pragma unroll
         for (int d0 = 0; d0 < Dp; d0 += 64) {
             const int d = d0 + ty * 4;
             if (d >= Dp) break;
-            float acc[4][4];
+            float s[4][4];
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int u = 0; u < 4; ++u) acc[i][u] = 0.f;
-#pragma unroll 4
+                for (int u = 0; u < 4; ++u) s[i][u] = 0.f;
+#pragma unroll 2
             for (int j = 0; j < DL_C; ++j) {
-                const float4 k = *reinterpret_cast<const float4*>(K + j * Ds + d), b = *reinterpret_cast<const float4*>(B + j * Ds + d);
-                const float4 v = *reinterpret_cast<const float4*>(Vs + j * 68 + tx * 4), y = *reinterpret_cast<const float4*>(Ys + j * 68 + tx * 4);
+                const float4 k = ld4(K + j * Ds + d), b = ld4(B + j * Ds + d), v = ld4(Vs + j * DL_VS + tx * 4), y = ld4(Ys + j * DL_VS + tx * 4);
                 const float kk[4] = {k.x, k.y, k.z, k.w}, bb[4] = {b.x, b.y, b.z, b.w}, vv[4] = {v.x, v.y, v.z, v.w}, yy[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
-                    for (int u = 0; u < 4; ++u) acc[i][u] = fmaf(kk[i], vv[u], fmaf(-bb[i], yy[u], acc[i][u]));
+                    for (int u = 0; u < 4; ++u) s[i][u] = fmaf(kk[i], vv[u], fmaf(-bb[i], yy[u], s[i][u]));
             }
-            if (v0 + tx * 4 < rec.Vp) {
+            if (v0 + tx * 4 < Vp) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const float w = wc[d + i];
-                    *reinterpret_cast<float4*>(out + rec.u() + (int64_t)(d + i) * rec.Vp + v0 + tx * 4) = make_float4(acc[i][0] * w, acc[i][1] * w, acc[i][2] * w, acc[i][3] * w);
+                    *reinterpret_cast<float4*>(out + rec.u() + (d + i) * Vp + v0 + tx * 4) = make_float4(s[i][0] * w, s[i][1] * w, s[i][2] * w, s[i][3] * w);
                 }
             }
         }
+        __syncthreads();
     }
 }
 
-// ---- pass B: grid (value tiles of DL_VT, H, B) -------------------------------------------------------------------------------------------
-// Dynamic shared memory: S [Dp][DL_SS] | two stages of (P' [C][Ds] | beta W_C [C][Ds] | W_C [Dp]) | Y [C][20]
-__host__ __device__ inline int delta_scan_floats(int D) {
-    const int Ds = delta_ds(D), Dp = (D + 3) & ~3;
-    return ((Dp * DL_SS + 3) & ~3) + 2 * (2 * DL_C * Ds + Dp) + DL_C * 20;
-}
+// ---- pass B: grid (value tiles of VT, H, B), 16 * VT threads ------------------------------------------------------------------------------------
+// Dynamic shared memory: S [Dp][VT + 2] | Y [C][YS] | NST stages of (P' [C][Ds] | beta W_C [C][Ds] | W_C [Dp] | the thread's own pieces of U)
+__host__ __device__ constexpr int delta_stage_floats(int D, int VT) { return 2 * DL_C * delta_ds(D) + delta_up4(D) + (delta_up4(D) + 63) / 64 * 64 * VT; }
+__host__ __device__ constexpr int delta_scan_floats(int D, int VT, int nst) { return delta_up4(delta_up4(D) * (VT + 2)) + DL_C * (VT == 16 ? 24 : 8) + nst * delta_stage_floats(D, VT); }
 
 __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
     const unsigned s = (unsigned)__cvta_generic_to_shared(dst);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(src));
 }
 
-template <int NU>   // key channels per thread row group: D <= 64 * NU
-__global__ void __launch_bounds__(DL_NT) delta_scan_kernel(const DeltaArgs a, const b200seq_step st) {
+template <int TD, int VT, int NST>
+__global__ void __launch_bounds__(16 * VT) delta_scan_kernel(const DeltaArgs a, const b200seq_step st) {
     extern __shared__ __align__(16) float sm[];
-    const int D = a.D, V = a.V, H = a.H, Ds = delta_ds(D), Dp = (D + 3) & ~3;
+    constexpr int NT = 16 * VT, SS = VT + 2, YS = VT == 16 ? 24 : 8;
+    const int D = TD ? TD : a.D, V = TD ? TD : a.V, H = a.H;
     const DeltaRec rec(D, V);
-    const int stage = 2 * DL_C * Ds + Dp;
+    const int Ds = rec.Ds, Dp = rec.Dp, Vp = rec.Vp;
+    const int nu = (Dp + 63) >> 6;                  // groups of 64 key channels
+    const int stage = 2 * DL_C * Ds + Dp + nu * 64 * VT;
     float* S = sm;
-    float* buf = S + ((Dp * DL_SS + 3) & ~3);
-    float* Y = buf + 2 * stage;
-    const int v0 = blockIdx.x * DL_VT, h = blockIdx.y, e = blockIdx.z, tid = threadIdx.x;
+    float* Y = S + ((Dp * SS + 3) & ~3);
+    float* buf = Y + DL_C * YS;
+    const int v0 = blockIdx.x * VT, h = blockIdx.y, e = blockIdx.z, tid = threadIdx.x;
     int c0 = 0;
     for (int i = 0; i < e; ++i) c0 += (st.ent_start[i + 1] - st.ent_start[i] + DL_C - 1) / DL_C;
     const int nc = (st.ent_start[e + 1] - st.ent_start[e] + DL_C - 1) / DL_C;
     if (nc == 0) return;
     float* slot = a.state + ((int64_t)st.ent_slot[e] * H + h) * D * V;
     const bool fresh = st.ent_pos0[e] == 0;
-    for (int it = tid; it < Dp * DL_VT; it += DL_NT) {
-        const int d = it / DL_VT, cc = it - d * DL_VT;
-        S[d * DL_SS + cc] = (!fresh && d < D && v0 + cc < V) ? slot[(int64_t)d * V + v0 + cc] : 0.f;
+    for (int it = tid; it < Dp * VT; it += NT) {
+        const int d = it / VT, cc = it - d * VT;
+        S[d * SS + cc] = (!fresh && d < D && v0 + cc < V) ? slot[(int64_t)d * V + v0 + cc] : 0.f;
     }
-    auto fetch = [&](int c, int s) {
-        const float* g = a.chunk + ((int64_t)(c0 + c) * H + h) * rec.size();
-        float* b = buf + s * stage;
-        const int q = Dp >> 2;
-        for (int it = tid; it < 2 * DL_C * q; it += DL_NT) {   // P' rows, then beta W_C rows: adjacent in the record
-            const int i = it / q, d4 = it - i * q;
-            cp_async16(b + i * Ds + 4 * d4, g + (int64_t)i * Dp + 4 * d4);
+    // Y = P' S: rows rg * 4 + i, columns cg * 2 + u; update: channels dgr * 4 + i (+ 64 n), columns vg * 4 + u; the four lanes kq share out the sums
+    const int kq = tid & 3, rest = tid >> 2, dgr = rest / (VT / 4), vg = rest % (VT / 4), rg = rest / (VT / 2), cg = rest % (VT / 2);
+    const bool vin = v0 + vg * 4 < Vp;
+    float* rec0 = a.chunk + ((int64_t)c0 * H + h) * rec.size();
+    const int64_t rstep = (int64_t)H * rec.size();
+    const int mine = (dgr * 4 + kq) * Vp + v0 + vg * 4;      // this thread's piece of U (channel dgr * 4 + kq + 64 n)
+    auto fetch = [&](int c) {
+        if (c < nc) {
+            const float* g = rec0 + c * rstep;
+            float* b = buf + (c % NST) * stage;
+            const int n16 = (2 * DL_C * Ds + Dp) >> 2;
+            for (int it = tid; it < n16; it += NT) cp_async16(b + 4 * it, g + 4 * it);
+            float* ub = b + 4 * n16;
+            for (int n = 0; n < nu; ++n)
+                if (vin && n * 64 + dgr * 4 < Dp) cp_async16(ub + 4 * (n * NT + tid), g + rec.u() + mine + n * 64 * Vp);
         }
-        for (int it = tid; it < q; it += DL_NT) cp_async16(b + 2 * DL_C * Ds + 4 * it, g + rec.w() + 4 * it);
         asm volatile("cp.async.commit_group;\n");
     };
-    // this thread's part of the update: channels dgr * 4 + kq (+ 64 per step), value columns vg * 4 .. + 3
-    const int kq = tid & 3, rest = tid >> 2, dgr = rest >> 2, vg = rest & 3;
-    const int rg = rest >> 3, cg = rest & 7;
-    const bool vin = v0 + vg * 4 < rec.Vp;
-    float4 un[NU];
-    auto load_u = [&](int c) {
-        const float* g = a.chunk + ((int64_t)(c0 + c) * H + h) * rec.size() + rec.u() + v0 + vg * 4;
 #pragma unroll
-        for (int n = 0; n < NU; ++n) {
-            const int d = n * 64 + dgr * 4 + kq;
-            un[n] = (vin && d < Dp) ? *reinterpret_cast<const float4*>(g + (int64_t)d * rec.Vp) : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
-    };
-    fetch(0, 0);
-    load_u(0);
+    for (int i = 0; i < NST - 1; ++i) fetch(i);
     for (int c = 0; c < nc; ++c) {
-        float4 uc[NU];
-#pragma unroll
-        for (int n = 0; n < NU; ++n) uc[n] = un[n];
-        if (c + 1 < nc) {
-            fetch(c + 1, (c + 1) & 1);
-            load_u(c + 1);
-            asm volatile("cp.async.wait_group 1;\n");
-        } else {
-            asm volatile("cp.async.wait_group 0;\n");
-        }
-        __syncthreads();   // stage c is in place, S is the state in front of chunk c
-        const float* Pm = buf + (c & 1) * stage;
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(NST - 2));
+        __syncthreads();   // stage c is in place, S is the state in front of chunk c, the stage of chunk c - 1 is free
+        fetch(c + NST - 1);
+        const float* Pm = buf + (c % NST) * stage;
         const float* Bm = Pm + DL_C * Ds;
         const float* wc = Bm + DL_C * Ds;
-        {   // Y = P' S: rows rg * 4 + i, columns cg * 2 + u, key channels dealt to the four lanes kq
+        const float* ub = wc + Dp;
+        {
             float acc[4][2];
 #pragma unroll
             for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = 0.f;
+#pragma unroll 4
             for (int d = kq * 4; d < Dp; d += 16) {
                 float4 p[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) p[i] = *reinterpret_cast<const float4*>(Pm + (rg * 4 + i) * Ds + d);
+                for (int i = 0; i < 4; ++i) p[i] = ld4(Pm + (rg * 4 + i) * Ds + d);
 #pragma unroll
                 for (int dd = 0; dd < 4; ++dd) {
-                    const float2 s = *reinterpret_cast<const float2*>(S + (d + dd) * DL_SS + cg * 2);
+                    const float2 s = *reinterpret_cast<const float2*>(S + (d + dd) * SS + cg * 2);
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const float pv = dd == 0 ? p[i].x : dd == 1 ? p[i].y : dd == 2 ? p[i].z : p[i].w;
@@ -460,22 +513,27 @@ __global__ void __launch_bounds__(DL_NT) delta_scan_kernel(const DeltaArgs a, co
                     }
                 }
             }
-            float y0 = 0.f, y1 = 0.f;
+            // sum over the four lanes; lane kq keeps row kq
+            float m[2][2], f[2];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
+            for (int i = 0; i < 2; ++i)
 #pragma unroll
                 for (int u = 0; u < 2; ++u) {
-                    acc[i][u] += __shfl_xor_sync(0xffffffffu, acc[i][u], 1);
-                    acc[i][u] += __shfl_xor_sync(0xffffffffu, acc[i][u], 2);
+                    const float send = (kq & 2) ? acc[i][u] : acc[i + 2][u], keep = (kq & 2) ? acc[i + 2][u] : acc[i][u];
+                    m[i][u] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
                 }
-                if (kq == i) y0 = acc[i][0], y1 = acc[i][1];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const float send = (kq & 1) ? m[0][u] : m[1][u], keep = (kq & 1) ? m[1][u] : m[0][u];
+                f[u] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
             }
-            *reinterpret_cast<float2*>(Y + (rg * 4 + kq) * 20 + cg * 2) = make_float2(y0, y1);
+            *reinterpret_cast<float2*>(Y + (rg * 4 + kq) * YS + cg * 2) = make_float2(f[0], f[1]);
         }
         __syncthreads();
-        float* gz = a.chunk + ((int64_t)(c0 + c) * H + h) * rec.size() + rec.u() + v0 + vg * 4;
+        float* gz = rec0 + c * rstep + rec.u() + mine;
 #pragma unroll
-        for (int n = 0; n < NU; ++n) {   // S = W_C S + U - (beta W_C)^T Y; the old S takes U's place in the record
+        for (int n = 0; n < (TD ? TD / 64 : 4); ++n) {   // S = W_C S + U - (beta W_C)^T Y; the old S takes U's place in the record
+            if (n >= nu) break;
             const int db = n * 64 + dgr * 4;
             const bool dok = db < Dp;    // Dp is a multiple of 4: all four channels or none (the same for the four lanes kq)
             float acc[4][4];
@@ -485,8 +543,9 @@ __global__ void __launch_bounds__(DL_NT) delta_scan_kernel(const DeltaArgs a, co
                 for (int u = 0; u < 4; ++u) acc[i][u] = 0.f;
             if (dok) {
 #pragma unroll
-                for (int j = kq; j < DL_C; j += 4) {
-                    const float4 b = *reinterpret_cast<const float4*>(Bm + j * Ds + db), y = *reinterpret_cast<const float4*>(Y + j * 20 + vg * 4);
+                for (int jj = 0; jj < DL_C / 4; ++jj) {
+                    const int j = 4 * jj + kq;
+                    const float4 b = ld4(Bm + j * Ds + db), y = ld4(Y + j * YS + vg * 4);
                     const float bb[4] = {b.x, b.y, b.z, b.w}, yy[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
                     for (int i = 0; i < 4; ++i)
@@ -500,77 +559,80 @@ __global__ void __launch_bounds__(DL_NT) delta_scan_kernel(const DeltaArgs a, co
             for (int i = 0; i < 2; ++i)
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
-                    const float send = (kq & 2) ? acc[i][u] : acc[i + 2][u], mine = (kq & 2) ? acc[i + 2][u] : acc[i][u];
-                    m[i][u] = mine + __shfl_xor_sync(0xffffffffu, send, 2);
+                    const float send = (kq & 2) ? acc[i][u] : acc[i + 2][u], keep = (kq & 2) ? acc[i + 2][u] : acc[i][u];
+                    m[i][u] = keep + __shfl_xor_sync(0xffffffffu, send, 2);
                 }
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const float send = (kq & 1) ? m[0][u] : m[1][u], mine = (kq & 1) ? m[1][u] : m[0][u];
-                f[u] = mine + __shfl_xor_sync(0xffffffffu, send, 1);
+                const float send = (kq & 1) ? m[0][u] : m[1][u], keep = (kq & 1) ? m[1][u] : m[0][u];
+                f[u] = keep + __shfl_xor_sync(0xffffffffu, send, 1);
             }
             if (dok) {
                 const int d = db + kq;
-                float2* sp = reinterpret_cast<float2*>(S + d * DL_SS + vg * 4);
+                float2* sp = reinterpret_cast<float2*>(S + d * SS + vg * 4);
                 const float2 s0 = sp[0], s1 = sp[1];
-                if (vin) *reinterpret_cast<float4*>(gz + (int64_t)d * rec.Vp) = make_float4(s0.x, s0.y, s1.x, s1.y);
+                float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (vin) {
+                    u = ld4(ub + 4 * (n * NT + tid));
+                    *reinterpret_cast<float4*>(gz + n * 64 * Vp) = make_float4(s0.x, s0.y, s1.x, s1.y);
+                }
                 const float w = wc[d];
-                sp[0] = make_float2(fmaf(w, s0.x, uc[n].x - f[0]), fmaf(w, s0.y, uc[n].y - f[1]));
-                sp[1] = make_float2(fmaf(w, s1.x, uc[n].z - f[2]), fmaf(w, s1.y, uc[n].w - f[3]));
+                sp[0] = make_float2(fmaf(w, s0.x, u.x - f[0]), fmaf(w, s0.y, u.y - f[1]));
+                sp[1] = make_float2(fmaf(w, s1.x, u.z - f[2]), fmaf(w, s1.y, u.w - f[3]));
             }
         }
-        __syncthreads();   // S is complete; the stage of chunk c may be refilled
     }
-    for (int it = tid; it < D * DL_VT; it += DL_NT) {
-        const int d = it / DL_VT, cc = it - d * DL_VT;
-        if (v0 + cc < V) slot[(int64_t)d * V + v0 + cc] = S[d * DL_SS + cc];
+    __syncthreads();
+    for (int it = tid; it < D * VT; it += NT) {
+        const int d = it / VT, cc = it - d * VT;
+        if (v0 + cc < V) slot[(int64_t)d * V + v0 + cc] = S[d * SS + cc];
     }
 }
 
 // ---- pass C: grid (chunks, H), 128 threads; thread (ty, tx): tokens ty * 4 + i, value columns tx * 4 + u of a tile of 64 --------------------
-// Dynamic shared memory: R' [C][Ds] | slab of the start state [32][68] | o [C][Vp + 4]
-constexpr int DL_NC = 128;
-__host__ __device__ inline int delta_out_floats(int D, int V) { return DL_C * delta_ds(D) + 32 * 68 + DL_C * (((V + 3) & ~3) + 4); }
+// Dynamic shared memory: R' [C][Ds] | slab of the start state [64][VS] | o [C][Vp + 4]
+constexpr int DL_NC = 128, DL_ZS = 64;
+__host__ __device__ constexpr int delta_out_floats(int D, int V) { return DL_C * delta_ds(D) + DL_ZS * DL_VS + DL_C * (delta_up4(V) + 4); }
 
+template <int TD>
 __global__ void __launch_bounds__(DL_NC) delta_out_kernel(const DeltaArgs a, const b200seq_step st) {
     extern __shared__ __align__(16) float sm[];
-    const int D = a.D, V = a.V, H = a.H, Ds = delta_ds(D), Dp = (D + 3) & ~3;
+    const int D = TD ? TD : a.D, V = TD ? TD : a.V, H = a.H;
     const DeltaRec rec(D, V);
-    const int Os = rec.Vp + 4;
-    float *R = sm, *Z = R + DL_C * Ds, *O = Z + 32 * 68;
+    const int Ds = rec.Ds, Dp = rec.Dp, Vp = rec.Vp, Os = Vp + 4;
+    float *R = sm, *Z = R + DL_C * Ds, *O = Z + DL_ZS * DL_VS;
     const int c = blockIdx.x, h = blockIdx.y;
     int e, row0, len;
     if (!find_chunk(st, c, DL_C, e, row0, len)) return;
     const float* g = a.chunk + ((int64_t)c * H + h) * rec.size();
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int q = Dp >> 2;
-    for (int it = tid; it < DL_C * q; it += DL_NC) {
-        const int i = it / q, d4 = it - i * q;
-        *reinterpret_cast<float4*>(R + i * Ds + 4 * d4) = *reinterpret_cast<const float4*>(g + rec.r() + (int64_t)i * Dp + 4 * d4);
-    }
+    for (int it = tid; it < DL_C * Ds / 4; it += DL_NC) cp_async16(R + 4 * it, g + rec.r() + 4 * it);
     for (int v0 = 0; v0 < V; v0 += 64) {
         float acc[4][4];
-        const bool vin = v0 + tx * 4 < rec.Vp;
+        const bool vin = v0 + tx * 4 < Vp;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const float4 o = vin ? *reinterpret_cast<const float4*>(g + rec.o() + (int64_t)(ty * 4 + i) * rec.Vp + v0 + tx * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 o = vin ? ld4(g + rec.o() + (ty * 4 + i) * Vp + v0 + tx * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
             acc[i][0] = o.x, acc[i][1] = o.y, acc[i][2] = o.z, acc[i][3] = o.w;
         }
-        for (int d0 = 0; d0 < Dp; d0 += 32) {
+        for (int d0 = 0; d0 < Dp; d0 += DL_ZS) {
             __syncthreads();
-            for (int it = tid; it < 32 * 16; it += DL_NC) {
+            for (int it = tid; it < DL_ZS * 16; it += DL_NC) {
                 const int dd = it >> 4, c4 = it & 15;
-                *reinterpret_cast<float4*>(Z + dd * 68 + 4 * c4) = (d0 + dd < Dp && v0 + 4 * c4 < rec.Vp)
-                    ? *reinterpret_cast<const float4*>(g + rec.u() + (int64_t)(d0 + dd) * rec.Vp + v0 + 4 * c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (d0 + dd < Dp && v0 + 4 * c4 < Vp) cp_async16(Z + dd * DL_VS + 4 * c4, g + rec.u() + (d0 + dd) * Vp + v0 + 4 * c4);
             }
+            asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;\n");
             __syncthreads();
-            const int dn = min(32, Dp - d0);
+            if (!vin) continue;          // (columns beyond the last are neither copied nor used)
+            const int dn = min(DL_ZS, Dp - d0);
+#pragma unroll 2
             for (int dd = 0; dd < dn; dd += 4) {
                 float4 r[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) r[i] = *reinterpret_cast<const float4*>(R + (ty * 4 + i) * Ds + d0 + dd);
+                for (int i = 0; i < 4; ++i) r[i] = ld4(R + (ty * 4 + i) * Ds + d0 + dd);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
-                    const float4 z = *reinterpret_cast<const float4*>(Z + (dd + k) * 68 + tx * 4);
+                    const float4 z = ld4(Z + (dd + k) * DL_VS + tx * 4);
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const float rv = k == 0 ? r[i].x : k == 1 ? r[i].y : k == 2 ? r[i].z : r[i].w;
@@ -597,6 +659,39 @@ __global__ void __launch_bounds__(DL_NC) delta_out_kernel(const DeltaArgs a, con
         const float* nw = a.norm_w + (int64_t)h * V;
         for (int v = lane; v < V; v += 32) store_act(a.out, a.out_dtype, (t * H + h) * V + v, o[v] * rinv * nw[v] * sigmoidf_acc(gate[v]));
     }
+}
+
+template <typename K>
+static cudaError_t delta_smem(K kernel, size_t bytes) {
+    return bytes > 48 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) : cudaSuccess;
+}
+
+template <int TD, int VT, int NST>
+static cudaError_t delta_scan_launch(const DeltaArgs& a, const b200seq_step& st, cudaStream_t cs) {
+    const size_t sb = (size_t)delta_scan_floats(a.D, VT, NST) * sizeof(float);
+    const cudaError_t e = delta_smem(delta_scan_kernel<TD, VT, NST>, sb);
+    if (e == cudaSuccess) delta_scan_kernel<TD, VT, NST><<<dim3((a.V + VT - 1) / VT, a.H, st.B), 16 * VT, sb, cs>>>(a, st);
+    return e;
+}
+
+template <int TD>
+static int delta_portions(const DeltaArgs& a, const b200seq_step& st, cudaStream_t cs) {
+    const int chunks = (st.T + DL_C - 1) / DL_C + st.B;   // upper bound of the step's chunk count
+    const size_t sa = (size_t)delta_local_floats(a.D) * sizeof(float), sc = (size_t)delta_out_floats(a.D, a.V) * sizeof(float);
+    cudaError_t err = delta_smem(delta_local_kernel<TD>, sa);
+    if (err == cudaSuccess) err = delta_smem(delta_out_kernel<TD>, sc);
+    if (err != cudaSuccess) return cuda_status(err, "delta attribute");
+    delta_local_kernel<TD><<<dim3(chunks, a.H), DL_NT, sa, cs>>>(a, st);
+    SEQ_LAUNCH_CHECK("delta local pass");
+    // narrower value tiles while the wider ones would leave SMs idle
+    const bool narrow = (int64_t)a.H * st.B * ((a.V + 15) / 16) < 128;
+    if (TD == 0) err = a.D <= 128 ? delta_scan_launch<TD, 16, 3>(a, st, cs) : delta_scan_launch<TD, 16, 2>(a, st, cs);
+    else err = narrow ? delta_scan_launch<TD, 8, 3>(a, st, cs) : delta_scan_launch<TD, 16, 3>(a, st, cs);
+    if (err != cudaSuccess) return cuda_status(err, "delta attribute");
+    SEQ_LAUNCH_CHECK("delta scan pass");
+    delta_out_kernel<TD><<<dim3(chunks, a.H), DL_NC, sc, cs>>>(a, st);
+    SEQ_LAUNCH_CHECK("delta output pass");
+    return 0;
 }
 
 }  // namespace b200seq
@@ -636,30 +731,9 @@ extern "C" int b200seq_delta(const float* proj, int64_t ld, const b200seq_step* 
     const size_t need = b200seq_delta_scratch_floats(st->T, st->B, d->H, d->D, d->V);
     if (!wz || ldw < (int64_t)d->H * d->D) return fail(B200SEQ_ERR_INVALID_ARG, "delta: a step of portions needs the low-rank branch's rows");
     if (!scratch || scratch_floats < need || (reinterpret_cast<uintptr_t>(scratch) & 15)) return fail(B200SEQ_ERR_INVALID_ARG, "delta: a step of portions needs %zu floats of 16-byte aligned work area", need);
-    const int chunks = (st->T + DL_C - 1) / DL_C + st->B;   // upper bound of the step's chunk count
-    const size_t sa = (size_t)delta_local_floats(d->D) * sizeof(float), sb = (size_t)delta_scan_floats(d->D) * sizeof(float), sc = (size_t)delta_out_floats(d->D, d->V) * sizeof(float);
-    if (d->D > 256 || sa > 220 * 1024 || sb > 220 * 1024 || sc > 220 * 1024) return fail(B200SEQ_ERR_UNSUPPORTED, "delta: head sizes too large");
-    cudaError_t err = cudaSuccess;
-    static size_t set_a = 48 * 1024, set_c = 48 * 1024;
-    if (sa > set_a) err = cudaFuncSetAttribute(delta_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sa), set_a = sa;
-    if (err == cudaSuccess && sc > set_c) err = cudaFuncSetAttribute(delta_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sc), set_c = sc;
-    if (err != cudaSuccess) return cuda_status(err, "delta attribute");
-    delta_local_kernel<<<dim3(chunks, d->H), DL_NT, sa, cs>>>(a, *st);
-    SEQ_LAUNCH_CHECK("delta local pass");
-    const dim3 gb((d->V + DL_VT - 1) / DL_VT, d->H, st->B);
-#define DELTA_SCAN(NU_)                                                                                                          \
-    do {                                                                                                                         \
-        static size_t set_ = 48 * 1024;                                                                                          \
-        if (sb > set_) err = cudaFuncSetAttribute(delta_scan_kernel<NU_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sb), set_ = sb; \
-        if (err == cudaSuccess) delta_scan_kernel<NU_><<<gb, DL_NT, sb, cs>>>(a, *st);                                           \
-    } while (0)
-    if (d->D <= 64) DELTA_SCAN(1);
-    else if (d->D <= 128) DELTA_SCAN(2);
-    else DELTA_SCAN(4);
-#undef DELTA_SCAN
-    if (err != cudaSuccess) return cuda_status(err, "delta attribute");
-    SEQ_LAUNCH_CHECK("delta scan pass");
-    delta_out_kernel<<<dim3(chunks, d->H), DL_NC, sc, cs>>>(a, *st);
-    SEQ_LAUNCH_CHECK("delta output pass");
-    return 0;
+    if (d->D > 256 || (size_t)delta_local_floats(d->D) * 4 > 220 * 1024 || (size_t)delta_out_floats(d->D, d->V) * 4 > 220 * 1024)
+        return fail(B200SEQ_ERR_UNSUPPORTED, "delta: head sizes too large");
+    if (d->D == 64 && d->V == 64) return delta_portions<64>(a, *st, cs);
+    if (d->D == 128 && d->V == 128) return delta_portions<128>(a, *st, cs);
+    return delta_portions<0>(a, *st, cs);
 }
