@@ -2,6 +2,8 @@
 // positions that enter as a sinusoid at the embedding, rows added in front of a looped span of layers, and an addition per layer that
 // depends on the token id.  Between two sublayers ONE kernel: norm of the sublayer's result, residual sum, additions, the next sublayer's
 // norm, its input in the activation type.  All arithmetic in f32.
+#include <cooperative_groups.h>
+
 #include "seq_common.cuh"
 
 namespace b200seq {
@@ -33,6 +35,7 @@ struct EmbedPos {
     float eps;
     void* a;                // or null
     int a_dtype;
+    int pairs;
 };
 __global__ void embed_pos_kernel(const EmbedPos p, const b200seq_step st) {
     extern __shared__ __align__(16) float row[];   // [W] | 40 of reduction scratch
@@ -43,6 +46,17 @@ __global__ void embed_pos_kernel(const EmbedPos p, const b200seq_step st) {
     for (int i = threadIdx.x; i < np; i += blockDim.x) {
         float sn = 0.f, cs = 0.f;
         if (p.freq) sincos_pos(pos, p.freq[i], p.freq[np + i], sn, cs);
+        if (p.pairs) {   // even width, aligned rows: both elements of a pair in one access
+            const float2 tv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(src + 2 * i));
+            float2 v = make_float2(fmaf(tv.x, p.scale, sn), fmaf(tv.y, p.scale, cs));
+            const int64_t o = (int64_t)t * W + 2 * i;
+            if (p.x0) *reinterpret_cast<float2*>(p.x0 + o) = v;
+            if (p.add_vec) v.x += p.add_vec[2 * i], v.y += p.add_vec[2 * i + 1];
+            *reinterpret_cast<float2*>(p.x + o) = v;
+            *reinterpret_cast<float2*>(row + 2 * i) = v;
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
+            continue;
+        }
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const int j = 2 * i + k;
@@ -162,15 +176,15 @@ __global__ void __launch_bounds__(512) sandwich_norm_reg_kernel(const SandwichAr
 
 // ---- the addition that depends on the token id ---------------------------------------------------------------------------------------------------
 // g[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][col + j]
-__global__ void token_gate_kernel(const float* __restrict__ z, int64_t ldz, int T, int dim, const __nv_bfloat16* __restrict__ table, int64_t ldt, int col,
+// grid (T)
+__global__ void token_gate_kernel(const float* __restrict__ z, int64_t ldz, int dim, const __nv_bfloat16* __restrict__ table, int64_t ldt, int col,
                                   const int32_t* __restrict__ ids, void* __restrict__ out, int out_dtype) {
-    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (int64_t)T * dim) return;
-    const int t = (int)(i / dim), j = (int)(i - (int64_t)t * dim);
-    store_act(out, out_dtype, i, gelu_tanhf_acc(z[t * ldz + j]) * __bfloat162float(table[(int64_t)ids[t] * ldt + col + j]));
+    const int t = blockIdx.x;
+    const __nv_bfloat16* row = table + (int64_t)ids[t] * ldt + col;
+    for (int j = threadIdx.x; j < dim; j += blockDim.x) store_act(out, out_dtype, (int64_t)t * dim + j, gelu_tanhf_acc(z[t * ldz + j]) * __bfloat162float(row[j]));
 }
 
-// Steps of few tokens: the norm of the sublayer's result, the residual sum, the token's addition and the next norm in one kernel, a block per row r
+// Steps of few tokens: the norm of the sublayer's result, the residual sum, the token's addition and the next norm in one kernel.  Any sizes: a block per row r
 // (token t = rows ? rows[r] : r).  Dynamic shared memory: x [W] | projected addition [W] | gated [dim] | 40
 struct SideArgs {
     SandwichArgs s;                   // x, y, w: the sublayer this closes; add_row / add_vec / fin_w / outputs: after the addition
@@ -186,7 +200,6 @@ __device__ __forceinline__ void bf8(const uint4 v, float* f) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) f[2 * i] = __uint_as_float(u[i] << 16), f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
 }
-template <bool VEC>
 __global__ void __launch_bounds__(1024) side_close_kernel(const SideArgs p) {
     extern __shared__ __align__(16) float sm[];
     const SandwichArgs& a = p.s;
@@ -208,18 +221,7 @@ __global__ void __launch_bounds__(1024) side_close_kernel(const SideArgs p) {
     for (int j = wid; j < dim; j += nw) {
         const __nv_bfloat16* wr = p.gate + (int64_t)j * W;
         float acc = 0.f;
-        if (VEC) {
-#pragma unroll 4
-            for (int k = lane * 8; k < W; k += 256) {
-                float f[8];
-                bf8(__ldg(reinterpret_cast<const uint4*>(wr + k)), f);
-                const float4 u0 = *reinterpret_cast<const float4*>(x + k), u1 = *reinterpret_cast<const float4*>(x + k + 4);
-                acc = fmaf(f[0], u0.x, fmaf(f[1], u0.y, fmaf(f[2], u0.z, fmaf(f[3], u0.w, acc))));
-                acc = fmaf(f[4], u1.x, fmaf(f[5], u1.y, fmaf(f[6], u1.z, fmaf(f[7], u1.w, acc))));
-            }
-        } else {
-            for (int k = lane; k < W; k += 32) acc = fmaf(__bfloat162float(wr[k]), x[k], acc);
-        }
+        for (int k = lane; k < W; k += 32) acc = fmaf(__bfloat162float(wr[k]), x[k], acc);
         acc = warp_sum(acc);
         if (lane == 0) g[j] = gelu_tanhf_acc(acc) * __bfloat162float(tab[j]);
     }
@@ -228,16 +230,7 @@ __global__ void __launch_bounds__(1024) side_close_kernel(const SideArgs p) {
     for (int i = tid; i < W; i += nt) {
         const __nv_bfloat16* wr = p.proj + (int64_t)i * dim;
         float acc = 0.f;
-        if (VEC) {
-            for (int j = 0; j < dim; j += 8) {
-                float f[8];
-                bf8(__ldg(reinterpret_cast<const uint4*>(wr + j)), f);
-#pragma unroll
-                for (int u = 0; u < 8; ++u) acc = fmaf(f[u], g[j + u], acc);
-            }
-        } else {
-            for (int j = 0; j < dim; ++j) acc = fmaf(__bfloat162float(wr[j]), g[j], acc);
-        }
+        for (int j = 0; j < dim; ++j) acc = fmaf(__bfloat162float(wr[j]), g[j], acc);
         y2[i] = acc;
         ss = fmaf(acc, acc, ss);
     }
@@ -255,6 +248,104 @@ __global__ void __launch_bounds__(1024) side_close_kernel(const SideArgs p) {
     float rf = 1.f;
     if (a.fin_w) rf = 1.0f / sqrtf(block_sum(sf, red) / (float)W + a.eps);
     for (int i = tid; i < W; i += nt) store_act(a.a_out, a.out_dtype, (int64_t)r * W + i, a.fin_w ? x[i] * rf * a.fin_w[i] : x[i]);
+}
+
+// The same with a cluster of SC_CL blocks per row, each of which streams its share of both projections: the gate's rows are dealt to the blocks (their
+// results go to every block's shared memory), then every block has a slice of the model width.  W % 8 == 0 and dim % 8 == 0.
+// Dynamic shared memory: x [W] | projected addition [slice] | gated [dim] | partial sums 2 x [SC_CL] | 40
+constexpr int SC_CL = 8, SC_NT = 256;
+__host__ __device__ constexpr int side_slice(int W) { return (W + SC_CL * 8 - 1) / (SC_CL * 8) * 8; }
+__global__ void __launch_bounds__(SC_NT) side_close_cluster_kernel(const SideArgs p) {
+    extern __shared__ __align__(16) float sm[];
+    namespace cg = cooperative_groups;
+    cg::cluster_group cl = cg::this_cluster();
+    const SandwichArgs& a = p.s;
+    const int W = a.W, dim = p.dim, tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
+    const int cr = (int)cl.block_rank(), ws = side_slice(W), w0 = cr * ws, w1 = min(W, w0 + ws);
+    float *x = sm, *y2 = x + W, *g = y2 + ws, *part = g + dim, *red = part + 2 * SC_CL;
+    const int r = blockIdx.x / SC_CL;
+    const int64_t t = a.rows ? a.rows[r] : r;
+    const float* y = a.y + t * W;
+    float ss = 0.f;
+    for (int i = tid * 4; i < W; i += SC_NT * 4) ss = sq4(ld4(y + i), ss);
+    const float rn = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
+    for (int i = tid * 4; i < W; i += SC_NT * 4) {
+        const float4 yv = ld4(y + i), w = ld4(a.w + i);
+        float4 xv = ld4(a.x + t * W + i);
+        xv.x += yv.x * rn * w.x, xv.y += yv.y * rn * w.y, xv.z += yv.z * rn * w.z, xv.w += yv.w * rn * w.w;
+        *reinterpret_cast<float4*>(x + i) = xv;
+    }
+    __syncthreads();
+    cl.sync();   // every block of the cluster runs: its shared memory may be written from now on (and no block has read this row's x_out place after it changed)
+    const __nv_bfloat16* tab = p.table + (int64_t)p.ids[t] * p.ldt + p.col;
+    for (int j = cr * (SC_NT / 32) + wid; j < dim; j += SC_CL * (SC_NT / 32)) {
+        const __nv_bfloat16* wr = p.gate + (int64_t)j * W;
+        float acc = 0.f;
+#pragma unroll 4
+        for (int k = lane * 8; k < W; k += 256) {
+            float f[8];
+            bf8(__ldg(reinterpret_cast<const uint4*>(wr + k)), f);
+            const float4 u0 = ld4(x + k), u1 = ld4(x + k + 4);
+            acc = fmaf(f[0], u0.x, fmaf(f[1], u0.y, fmaf(f[2], u0.z, fmaf(f[3], u0.w, acc))));
+            acc = fmaf(f[4], u1.x, fmaf(f[5], u1.y, fmaf(f[6], u1.z, fmaf(f[7], u1.w, acc))));
+        }
+        acc = warp_sum(acc);
+        const float v = gelu_tanhf_acc(acc) * __bfloat162float(tab[j]);
+        if (lane < SC_CL) cl.map_shared_rank(g, lane)[j] = v;
+    }
+    cl.sync();
+    // eight lanes per row of the projection
+    const int sub = lane & 7;
+    ss = 0.f;
+    for (int i0 = w0 + wid * 4; i0 < w1; i0 += SC_NT / 32 * 4) {
+        const int i = i0 + (lane >> 3);
+        float acc = 0.f;
+        if (i < w1) {
+            const __nv_bfloat16* wr = p.proj + (int64_t)i * dim;
+#pragma unroll 4
+            for (int j = sub * 8; j < dim; j += 64) {
+                float f[8];
+                bf8(__ldg(reinterpret_cast<const uint4*>(wr + j)), f);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) acc = fmaf(f[u], g[j + u], acc);
+            }
+        }
+        acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+        acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+        acc += __shfl_xor_sync(0xffffffffu, acc, 4);
+        if (i < w1 && sub == 0) {
+            y2[i - w0] = acc;
+            ss = fmaf(acc, acc, ss);
+        }
+    }
+    ss = block_sum(ss, red);
+    if (tid < SC_CL) cl.map_shared_rank(part, tid)[cr] = ss;
+    cl.sync();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < SC_CL; ++i) ss += part[i];
+    const float r2 = 1.0f / sqrtf(ss / (float)W + a.eps);
+    float sf = 0.f;
+    for (int i = w0 + tid; i < w1; i += SC_NT) {
+        float xn = x[i] + y2[i - w0] * r2 * p.side_w[i];
+        if (a.add_row) xn += a.add_row[t * W + i];
+        if (a.add_vec) xn += a.add_vec[i];
+        x[i] = xn;
+        sf = fmaf(xn, xn, sf);
+        if (a.x_out) a.x_out[t * W + i] = xn;
+    }
+    if (!a.a_out) return;
+    float rf = 1.f;
+    if (a.fin_w) {
+        sf = block_sum(sf, red);
+        if (tid < SC_CL) cl.map_shared_rank(part, tid)[SC_CL + cr] = sf;
+        cl.sync();
+        sf = 0.f;
+#pragma unroll
+        for (int i = 0; i < SC_CL; ++i) sf += part[SC_CL + i];
+        rf = 1.0f / sqrtf(sf / (float)W + a.eps);
+    }
+    for (int i = w0 + tid; i < w1; i += SC_NT) store_act(a.a_out, a.out_dtype, (int64_t)r * W + i, a.fin_w ? x[i] * rf * a.fin_w[i] : x[i]);   // own elements only
 }
 
 }  // namespace b200seq
@@ -275,7 +366,8 @@ int b200seq_embed_pos(const void* table_bf16, const int32_t* ids, const b200seq_
         const cudaError_t e = cudaFuncSetAttribute(embed_pos_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return cuda_status(e, "embed_pos attribute");
     }
-    const EmbedPos p{(const __nv_bfloat16*)table_bf16, ids, freq, scale, W, x0, add_vec, x, fin_w, eps, a, a_dtype};
+    const EmbedPos p{(const __nv_bfloat16*)table_bf16, ids, freq, scale, W, x0, add_vec, x, fin_w, eps, a, a_dtype,
+                     W % 2 == 0 && ((reinterpret_cast<uintptr_t>(table_bf16) & 3) | (reinterpret_cast<uintptr_t>(x) & 7) | (reinterpret_cast<uintptr_t>(x0) & 7)) == 0};
     embed_pos_kernel<<<st->T, W >= 1024 ? 512 : 128, smem, (cudaStream_t)stream>>>(p, *st);
     SEQ_LAUNCH_CHECK("embed_pos");
     return 0;
@@ -321,8 +413,7 @@ int b200seq_token_gate(const float* z, int64_t ldz, int T, int dim, const void* 
     if (!z || !table_bf16 || !ids || !out || T < 0 || dim < 1 || col < 0 || ldz < dim || ldt < col + dim || !act_ok(out_dtype))
         return fail(B200SEQ_ERR_INVALID_ARG, "token_gate: bad arguments");
     if (T == 0) return 0;
-    const int64_t n = (int64_t)T * dim;
-    token_gate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(z, ldz, T, dim, (const __nv_bfloat16*)table_bf16, ldt, col, ids, out, out_dtype);
+    token_gate_kernel<<<T, dim <= 64 ? 64 : 128, 0, (cudaStream_t)stream>>>(z, ldz, dim, (const __nv_bfloat16*)table_bf16, ldt, col, ids, out, out_dtype);
     SEQ_LAUNCH_CHECK("token_gate");
     return 0;
 }
@@ -339,14 +430,29 @@ int b200seq_side_close(const float* x, const float* y, const float* w, float eps
     const SideArgs p{SandwichArgs{x, y, w, eps, add_row, add_vec, W, rows, x_out, a_out, out_dtype, fin_w}, (const __nv_bfloat16*)gate_bf16,
                      (const __nv_bfloat16*)proj_bf16, (const __nv_bfloat16*)table_bf16, ldt, col, dim, ids, side_w};
     const bool vec = W % 8 == 0 && dim % 8 == 0 && ((reinterpret_cast<uintptr_t>(gate_bf16) | reinterpret_cast<uintptr_t>(proj_bf16)) & 15) == 0;
+    auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    if (vec && R <= 65535 / SC_CL && al(x) && al(y) && al(w)) {
+        const size_t cs = ((size_t)W + side_slice(W) + dim + 2 * SC_CL + 40) * sizeof(float);
+        if (cs > 48 * 1024) {
+            const cudaError_t e = cudaFuncSetAttribute(side_close_cluster_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)cs);
+            if (e != cudaSuccess) return cuda_status(e, "side_close attribute");
+        }
+        cudaLaunchConfig_t cfg{};
+        cudaLaunchAttribute at{};
+        at.id = cudaLaunchAttributeClusterDimension;
+        at.val.clusterDim.x = SC_CL, at.val.clusterDim.y = 1, at.val.clusterDim.z = 1;
+        cfg.gridDim = dim3(R * SC_CL), cfg.blockDim = dim3(SC_NT), cfg.dynamicSmemBytes = cs, cfg.stream = (cudaStream_t)stream, cfg.attrs = &at, cfg.numAttrs = 1;
+        const cudaError_t e = cudaLaunchKernelEx(&cfg, side_close_cluster_kernel, p);
+        if (e != cudaSuccess) return cuda_status(e, "side_close");
+        count_launch();
+        return 0;
+    }
     if (smem > 48 * 1024) {
-        const cudaError_t e = vec ? cudaFuncSetAttribute(side_close_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
-                                  : cudaFuncSetAttribute(side_close_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(side_close_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return cuda_status(e, "side_close attribute");
     }
     const int nt = W >= 1024 ? 1024 : (W >= 512 ? 512 : 256);
-    if (vec) side_close_kernel<true><<<R, nt, smem, (cudaStream_t)stream>>>(p);
-    else side_close_kernel<false><<<R, nt, smem, (cudaStream_t)stream>>>(p);
+    side_close_kernel<<<R, nt, smem, (cudaStream_t)stream>>>(p);
     SEQ_LAUNCH_CHECK("side_close");
     return 0;
 }

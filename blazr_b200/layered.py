@@ -1374,7 +1374,7 @@ class LayeredModel:
         if R and (not n or debug_layers is not None):
             ops.group_rmsnorm(x if R == T and debug_layers is None else x.index_select(0, want.long()), self.final_norm, 1, cfg.eps, ws.fin[:R])
 
-    SIDE_FUSED_ELEMS = 1 << 17      # few tokens: up to this many weights per projection the token-dependent addition runs in one block per token
+    SIDE_FUSED_ELEMS = 1 << 20      # few tokens: up to this many weights per projection the token-dependent addition is part of the closing kernel
 
     def _run_sandwich(self, ws: _Workspace, T: int, B: int, R: int, debug_layers: Optional[list]) -> None:
         """sublayers in sequence over one residual x (f32), each normed on both sides.  Between sublayers ONE kernel: the norm of the sublayer's
