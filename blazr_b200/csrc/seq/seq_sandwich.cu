@@ -253,7 +253,8 @@ __global__ void __launch_bounds__(1024) side_close_kernel(const SideArgs p) {
 // The same with a cluster of SC_CL blocks per row, each of which streams its share of both projections: the gate's rows are dealt to the blocks (their
 // results go to every block's shared memory), then every block has a slice of the model width.  W % 8 == 0 and dim % 8 == 0.
 // Dynamic shared memory: x [W] | projected addition [slice] | gated [dim] | partial sums 2 x [SC_CL] | 40
-constexpr int SC_CL = 8, SC_NT = 256;
+constexpr int SC_CL = 8, SC_NT = 512;
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 __host__ __device__ constexpr int side_slice(int W) { return (W + SC_CL * 8 - 1) / (SC_CL * 8) * 8; }
 __global__ void __launch_bounds__(SC_NT) side_close_cluster_kernel(const SideArgs p) {
     extern __shared__ __align__(16) float sm[];
@@ -265,6 +266,13 @@ __global__ void __launch_bounds__(SC_NT) side_close_cluster_kernel(const SideArg
     float *x = sm, *y2 = x + W, *g = y2 + ws, *part = g + dim, *red = part + 2 * SC_CL;
     const int r = blockIdx.x / SC_CL;
     const int64_t t = a.rows ? a.rows[r] : r;
+    // the weights do not depend on what runs before: the block's share of them is on its way to L2 while the norm is computed
+    const __nv_bfloat16* tab = p.table + (int64_t)p.ids[t] * p.ldt + p.col;
+    for (int j = cr * (SC_NT / 32) + wid; j < dim; j += SC_CL * (SC_NT / 32)) {
+        for (int k = lane * 64; k < W; k += 2048) prefetch_l2(p.gate + (int64_t)j * W + k);
+        if (lane == 0) prefetch_l2(tab + j);
+    }
+    for (int64_t k = (int64_t)w0 * dim + tid * 64; k < (int64_t)w1 * dim; k += SC_NT * 64) prefetch_l2(p.proj + k);
     const float* y = a.y + t * W;
     float ss = 0.f;
     for (int i = tid * 4; i < W; i += SC_NT * 4) ss = sq4(ld4(y + i), ss);
@@ -277,11 +285,11 @@ __global__ void __launch_bounds__(SC_NT) side_close_cluster_kernel(const SideArg
     }
     __syncthreads();
     cl.sync();   // every block of the cluster runs: its shared memory may be written from now on (and no block has read this row's x_out place after it changed)
-    const __nv_bfloat16* tab = p.table + (int64_t)p.ids[t] * p.ldt + p.col;
     for (int j = cr * (SC_NT / 32) + wid; j < dim; j += SC_CL * (SC_NT / 32)) {
         const __nv_bfloat16* wr = p.gate + (int64_t)j * W;
+        const float tv = __bfloat162float(tab[j]);
         float acc = 0.f;
-#pragma unroll 4
+#pragma unroll 8
         for (int k = lane * 8; k < W; k += 256) {
             float f[8];
             bf8(__ldg(reinterpret_cast<const uint4*>(wr + k)), f);
@@ -290,32 +298,37 @@ __global__ void __launch_bounds__(SC_NT) side_close_cluster_kernel(const SideArg
             acc = fmaf(f[4], u1.x, fmaf(f[5], u1.y, fmaf(f[6], u1.z, fmaf(f[7], u1.w, acc))));
         }
         acc = warp_sum(acc);
-        const float v = gelu_tanhf_acc(acc) * __bfloat162float(tab[j]);
+        const float v = gelu_tanhf_acc(acc) * tv;
         if (lane < SC_CL) cl.map_shared_rank(g, lane)[j] = v;
     }
     cl.sync();
-    // eight lanes per row of the projection
+    // eight lanes per row of the projection, four rows per lane at a time
     const int sub = lane & 7;
     ss = 0.f;
-    for (int i0 = w0 + wid * 4; i0 < w1; i0 += SC_NT / 32 * 4) {
-        const int i = i0 + (lane >> 3);
-        float acc = 0.f;
-        if (i < w1) {
-            const __nv_bfloat16* wr = p.proj + (int64_t)i * dim;
-#pragma unroll 4
-            for (int j = sub * 8; j < dim; j += 64) {
-                float f[8];
-                bf8(__ldg(reinterpret_cast<const uint4*>(wr + j)), f);
+    for (int i0 = w0 + wid * 16 + (lane >> 3); i0 - (lane >> 3) < w1; i0 += SC_NT / 32 * 16) {
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+        for (int j = sub * 8; j < dim; j += 64) {
+            uint4 v[4];
 #pragma unroll
-                for (int u = 0; u < 8; ++u) acc = fmaf(f[u], g[j + u], acc);
+            for (int q = 0; q < 4; ++q) v[q] = i0 + 4 * q < w1 ? __ldg(reinterpret_cast<const uint4*>(p.proj + (int64_t)(i0 + 4 * q) * dim + j)) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                float f[8];
+                bf8(v[q], f);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) acc[q] = fmaf(f[u], g[j + u], acc[q]);
             }
         }
-        acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-        acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-        acc += __shfl_xor_sync(0xffffffffu, acc, 4);
-        if (i < w1 && sub == 0) {
-            y2[i - w0] = acc;
-            ss = fmaf(acc, acc, ss);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            acc[q] += __shfl_xor_sync(0xffffffffu, acc[q], 1);
+            acc[q] += __shfl_xor_sync(0xffffffffu, acc[q], 2);
+            acc[q] += __shfl_xor_sync(0xffffffffu, acc[q], 4);
+            if (i0 + 4 * q < w1 && sub == 0) {
+                y2[i0 + 4 * q - w0] = acc[q];
+                ss = fmaf(acc[q], acc[q], ss);
+            }
         }
     }
     ss = block_sum(ss, red);
