@@ -385,7 +385,7 @@ def _cost(name: str, shapes, scal, scen: dict, kw: dict = None):
         T, ld = sh[0][0]
         wz = T * d.H * d.D * 4 if scen["prefill"] else d.H * d.D * d.rank * 2
         # u^T S, decay, removal, k v^T, S^T r of the plain recurrence (the chunked form's own products are not counted)
-        return T * (ld * 4 + d.H * d.V * kw.get("out_es", 2)) + wz + 2 * scen["entries"] * d.H * d.D * d.V * 4, 9.0 * T * d.H * d.D * d.V, "f32" if scen["prefill"] else "hbm"
+        return T * (ld * 4 + d.H * d.V * sh[-2][1]) + wz + 2 * scen["entries"] * d.H * d.D * d.V * 4, 9.0 * T * d.H * d.D * d.V, "f32" if scen["prefill"] else "hbm"
     if name == "sandwich_norm":   # x, the result and the added rows in; x and / or the activation rows out
         rows = kw["rows"][0][0] if isinstance(kw.get("rows"), tuple) else sh[0][0][0]
         W = sh[0][0][1]
