@@ -7,7 +7,7 @@
 
 namespace b200seq {
 
-int launch_linear_tc(const void* x_bf16, int64_t ldx, const void* w_bf16, int M, int N, int K, float* y, int64_t ldy, cudaStream_t st);
+int launch_linear_tc(const void* x_bf16, int64_t ldx, const void* w_bf16, int M, int N, int K, float* y, int64_t ldy, int silu_lo, int silu_hi, cudaStream_t st);
 bool linear_tc_usable(int x_dtype, int64_t ldx, int M, int N, int K, const void* x, const void* w);
 int launch_linear_tc_act(const void* x, int64_t ldx, const void* w, int M, int N, int K, const ActParams act, void* out, int out_dtype, int64_t ldo,
                          cudaStream_t st);
@@ -36,7 +36,9 @@ struct GateEpi {
     int out_dtype;
     int64_t ldo;
     ActParams act;
+    int silu_lo, silu_hi;   // plain product: the columns [silu_lo, silu_hi) of y pass silu
 };
+__device__ __forceinline__ float silu_range(float v, int n, int lo, int hi) { return (n >= lo && n < hi) ? siluf_acc(v) : v; }
 
 template <typename XT, int MB, bool VEC>
 __global__ void __launch_bounds__(256) linear_rows_kernel(const XT* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, int M, int N, int K,
@@ -102,8 +104,8 @@ __global__ void __launch_bounds__(256) linear_rows_kernel(const XT* __restrict__
                         if (two) store_act(ge.out, ge.out_dtype, (int64_t)(m0 + m) * ge.ldo + n0 + 1, act_plain(ge.act.kind, s1));
                     }
                 } else {
-                    y[(int64_t)(m0 + m) * ldy + n0] = s0;
-                    if (two) y[(int64_t)(m0 + m) * ldy + n0 + 1] = s1;
+                    y[(int64_t)(m0 + m) * ldy + n0] = silu_range(s0, n0, ge.silu_lo, ge.silu_hi);
+                    if (two) y[(int64_t)(m0 + m) * ldy + n0 + 1] = silu_range(s1, n0 + 1, ge.silu_lo, ge.silu_hi);
                 }
             }
         }
@@ -114,7 +116,7 @@ __global__ void __launch_bounds__(256) linear_rows_kernel(const XT* __restrict__
 constexpr int TM = 64, TN = 64, TK = 16;
 template <typename XT>
 __global__ void __launch_bounds__(256) linear_tiled_kernel(const XT* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, int M, int N, int K,
-                                                           float* __restrict__ y, int64_t ldy) {
+                                                           float* __restrict__ y, int64_t ldy, int silu_lo, int silu_hi) {
     __shared__ float xs[TK][TM + 4];
     __shared__ float ws[TK][TN + 4];
     const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
@@ -154,14 +156,14 @@ __global__ void __launch_bounds__(256) linear_tiled_kernel(const XT* __restrict_
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) y[(int64_t)m * ldy + n] = acc[i][j];
+            if (n < N) y[(int64_t)m * ldy + n] = silu_range(acc[i][j], n, silu_lo, silu_hi);
         }
     }
 }
 
 template <typename XT>
 static void launch_rows(const XT* x, int64_t ldx, const __nv_bfloat16* w, int M, int N, int K, float* y, int64_t ldy, cudaStream_t st,
-                        const GateEpi ge = GateEpi{nullptr, 0, 0, ActParams{0, 0.f, 0.f, 0.f}}) {
+                        const GateEpi ge) {
     const bool vec = K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 &&
                      (ldx * (int64_t)sizeof(XT)) % 16 == 0;
     const int rpw = ((ge.out && act_kind_gated(ge.act.kind)) || (N + 15) / 16 >= 4 * 148) ? 2 : 1;   // few rows: one per warp, so that every SM streams weights
@@ -184,6 +186,11 @@ static void launch_rows(const XT* x, int64_t ldx, const __nv_bfloat16* w, int M,
 using namespace b200seq;
 
 extern "C" int b200seq_linear(const void* x, int x_dtype, int64_t ldx, const void* w, int M, int N, int K, float* y, int64_t ldy, int path, void* stream) {
+    return b200seq_linear_silu(x, x_dtype, ldx, w, M, N, K, y, ldy, 0, 0, path, stream);
+}
+
+extern "C" int b200seq_linear_silu(const void* x, int x_dtype, int64_t ldx, const void* w, int M, int N, int K, float* y, int64_t ldy, int silu_lo, int silu_hi, int path,
+                                   void* stream) {
     if (!x || !w || !y || M < 0 || N < 1 || K < 1 || ldx < K || ldy < N) return fail(B200SEQ_ERR_INVALID_ARG, "linear: bad arguments");
     if (x_dtype != B200SEQ_F32 && x_dtype != B200SEQ_BF16) return fail(B200SEQ_ERR_INVALID_ARG, "linear: activation dtype");
     if (M == 0) return 0;
@@ -195,15 +202,16 @@ extern "C" int b200seq_linear(const void* x, int x_dtype, int64_t ldx, const voi
     }
     if (path == B200SEQ_PATH_TC) {
         if (!linear_tc_usable(x_dtype, ldx, M, N, K, x, w)) return fail(B200SEQ_ERR_UNSUPPORTED, "linear: the tensor-core path needs bf16 activations, K %% 8 == 0 and 16-byte aligned rows");
-        return launch_linear_tc(x, ldx, w, M, N, K, y, ldy, st);
+        return launch_linear_tc(x, ldx, w, M, N, K, y, ldy, silu_lo, silu_hi, st);
     }
     if (path == B200SEQ_PATH_ROWS) {
-        if (x_dtype == B200SEQ_F32) launch_rows((const float*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, st);
-        else launch_rows((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, st);
+        const GateEpi ge{nullptr, 0, 0, ActParams{0, 0.f, 0.f, 0.f}, silu_lo, silu_hi};
+        if (x_dtype == B200SEQ_F32) launch_rows((const float*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, st, ge);
+        else launch_rows((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, st, ge);
     } else if (path == B200SEQ_PATH_TILED) {
         dim3 grid((N + TN - 1) / TN, (M + TM - 1) / TM);
-        if (x_dtype == B200SEQ_F32) linear_tiled_kernel<<<grid, 256, 0, st>>>((const float*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy);
-        else linear_tiled_kernel<<<grid, 256, 0, st>>>((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy);
+        if (x_dtype == B200SEQ_F32) linear_tiled_kernel<<<grid, 256, 0, st>>>((const float*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, silu_lo, silu_hi);
+        else linear_tiled_kernel<<<grid, 256, 0, st>>>((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, M, N, K, y, ldy, silu_lo, silu_hi);
     } else {
         return fail(B200SEQ_ERR_INVALID_ARG, "linear: unknown path %d", path);
     }
@@ -221,7 +229,7 @@ extern "C" int b200seq_linear_act(const void* x, int x_dtype, int64_t ldx, const
     if (M == 0) return 0;
     const ActParams ap{act, limit, alpha, shift};
     if (M <= 8) {   // few tokens: the weight-streaming kernel (gated kinds: a warp's two rows are one (gate, up) pair)
-        const GateEpi ge{out, out_dtype, ldo, ap};
+        const GateEpi ge{out, out_dtype, ldo, ap, 0, 0};
         if (x_dtype == B200SEQ_F32) launch_rows((const float*)x, ldx, (const __nv_bfloat16*)w, M, N, K, nullptr, 0, (cudaStream_t)stream, ge);
         else launch_rows((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, M, N, K, nullptr, 0, (cudaStream_t)stream, ge);
         SEQ_LAUNCH_CHECK("linear_act rows");

@@ -102,6 +102,7 @@ struct TcParams {
     const int32_t* offs;   // grouped form: [E + 1] first row of every group; rows of group e use the weight rows e * N .. e * N + N - 1
     int E;
     int heads;             // per-head form (blockIdx.z = head e): every row goes through every head's weight rows e * N .., reading the columns
+    int silu_lo, silu_hi;  // EPI_NONE: the columns [silu_lo, silu_hi) pass silu
     int64_t ocol;          // e * K .. of its x row and writing the columns e * ocol .. of its output row
 };
 constexpr int EPI_NONE = 0, EPI_GATED = 1, EPI_PLAIN_ACT = 2;
@@ -200,6 +201,10 @@ __global__ void __launch_bounds__(128) linear_tc_kernel(const __grid_constant__ 
             tc_wait_ld();
             if (p.epi == EPI_NONE) {
                 if (n < p.N) {
+                    if (n >= p.silu_lo && n < p.silu_hi) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(siluf_acc(__uint_as_float(r[j])));
+                    }
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
                         if (m0 + c + j < m_end) p.y[(int64_t)(m0 + c + j) * p.ldy + oc0 + n] = __uint_as_float(r[j]);
@@ -279,8 +284,9 @@ bool linear_tc_usable(int x_dtype, int64_t ldx, int M, int N, int K, const void*
            encode_fn() != nullptr;
 }
 
-int launch_linear_tc(const void* x, int64_t ldx, const void* w, int M, int N, int K, float* y, int64_t ldy, cudaStream_t st) {
+int launch_linear_tc(const void* x, int64_t ldx, const void* w, int M, int N, int K, float* y, int64_t ldy, int silu_lo, int silu_hi, cudaStream_t st) {
     TcParams p{};
+    p.silu_lo = silu_lo, p.silu_hi = silu_hi;
     p.y = y, p.ldy = ldy, p.M = M, p.N = N, p.K = K, p.epi = EPI_NONE;
     return launch(x, ldx, w, p, st);
 }

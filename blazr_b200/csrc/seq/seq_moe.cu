@@ -37,8 +37,17 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int64_t l
 // choice of one token by one warp: zr = its E router logits; sm = 2 * E + groups floats of shared memory
 // kind 0: sigmoid scores; kind 1: soft-max over the E logits; kind 2: choice by the logits, weights = soft-max over the chosen ones.
 // corr (or null) is added to the scores for the choice only.
-__device__ __forceinline__ void route_token(const float* zr, float* sm, int t, int lane, int E, int groups, int keep, int top, int32_t* __restrict__ ids,
-                                            float* __restrict__ wts, int32_t* __restrict__ counts, int kind = 0, const float* __restrict__ corr = nullptr) {
+struct RouteRule {
+    int E, groups, keep, top, kind;
+    const float* corr;
+    int group_best;   // a group's score: 2 = sum of its two largest scores, 1 = the largest
+    int renorm;       // 1 = weights divided by their sum
+    float scale;      // what the weights are multiplied by
+};
+__device__ __forceinline__ void route_token(const float* zr, float* sm, int t, int lane, const RouteRule& rule, int32_t* __restrict__ ids, float* __restrict__ wts,
+                                            int32_t* __restrict__ counts) {
+    const int E = rule.E, groups = rule.groups, keep = rule.keep, top = rule.top, kind = rule.kind;
+    const float* corr = rule.corr;
     float* s = sm;            // [E] scores
     float* avail = sm + E;    // [E] choice scores; a chosen or excluded expert is marked by -inf
     float* gsc = avail + E;   // [groups]
@@ -78,7 +87,7 @@ __device__ __forceinline__ void route_token(const float* zr, float* sm, int t, i
                 if (v > a) b = a, a = v;
                 else if (v > b) b = v;
             }
-            gsc[g] = gs > 1 ? a + b : a;
+            gsc[g] = (gs > 1 && rule.group_best == 2) ? a + b : a;
         }
         __syncwarp();
         // the `keep` best groups stay: mark them by a negative score, then exclude the experts of every other group
@@ -122,16 +131,16 @@ __device__ __forceinline__ void route_token(const float* zr, float* sm, int t, i
         sum += best;
         __syncwarp();
     }
-    const float inv = 1.0f / (sum + 1e-20f);
+    const float inv = rule.renorm ? rule.scale / (sum + 1e-20f) : rule.scale;
     __syncwarp();
     for (int k = lane; k < top; k += 32) wts[(int64_t)t * top + k] *= inv;
 }
 
 // grid (T), one warp per token
-__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, int E, int groups, int keep, int top, int32_t* __restrict__ ids,
-                                 float* __restrict__ wts, int32_t* __restrict__ counts, int kind, const float* __restrict__ corr) {
+__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const RouteRule rule, int32_t* __restrict__ ids, float* __restrict__ wts,
+                                 int32_t* __restrict__ counts) {
     extern __shared__ float sm[];
-    route_token(z + (int64_t)blockIdx.x * ldz, sm, blockIdx.x, threadIdx.x, E, groups, keep, top, ids, wts, counts, kind, corr);
+    route_token(z + (int64_t)blockIdx.x * ldz, sm, blockIdx.x, threadIdx.x, rule, ids, wts, counts);
 }
 
 // choice by table: one thread per (token, choice)
@@ -158,8 +167,8 @@ __device__ __forceinline__ float ldx(const XT* p);
 // rows and any rows stacked behind them), z[t][n] = x[t] . w[n] goes to memory and to shared memory, then warp 0 makes the token's choice.
 template <typename XT, bool VEC>
 __global__ void __launch_bounds__(256) moe_router_rows_kernel(const XT* __restrict__ x, int64_t ldx_, const __nv_bfloat16* __restrict__ w, int NR, int K,
-                                                              float* __restrict__ z, int64_t ldz, int E, int groups, int keep, int top,
-                                                              int32_t* __restrict__ ids, float* __restrict__ wts, int kind, const float* __restrict__ corr) {
+                                                              float* __restrict__ z, int64_t ldz, const RouteRule rule, int32_t* __restrict__ ids,
+                                                              float* __restrict__ wts) {
     extern __shared__ float sm[];   // NR logits, then the choice's 2 * E + groups floats
     const int t = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const XT* xr = x + (int64_t)t * ldx_;
@@ -190,7 +199,7 @@ __global__ void __launch_bounds__(256) moe_router_rows_kernel(const XT* __restri
         }
     }
     __syncthreads();
-    if (wid == 0) route_token(sm, sm + NR, t, lane, E, groups, keep, top, ids, wts, nullptr, kind, corr);
+    if (wid == 0) route_token(sm, sm + NR, t, lane, rule, ids, wts, nullptr);
 }
 
 // grid (E), 256 threads: block e places the pairs of expert e behind those of the experts before it, in pair order
@@ -534,18 +543,34 @@ int b200seq_moe_route(const float* z, int64_t ldz, int T, int E, int groups, int
 
 int b200seq_moe_route_ex(const float* z, int64_t ldz, int T, int E, int groups, int keep, int top, int kind, const float* correction, int32_t* ids, float* wts,
                          int32_t* counts, void* stream) {
-    if (kind < 0 || kind > 2) return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: score kind 0 (sigmoid), 1 (soft-max) or 2 (soft-max over the chosen)");
+    const b200seq_route_desc d{E, groups, keep, top, kind, 2, 1, 1.f, correction};
+    return b200seq_moe_route_rule(z, ldz, T, &d, ids, wts, counts, stream);
+}
+
+static int route_rule(const b200seq_route_desc* d, RouteRule& r, const char* what) {
+    if (!d) return fail(B200SEQ_ERR_INVALID_ARG, "%s: bad arguments", what);
+    if (d->kind < 0 || d->kind > 2) return fail(B200SEQ_ERR_INVALID_ARG, "%s: score kind 0 (sigmoid), 1 (soft-max) or 2 (soft-max over the chosen)", what);
+    if (d->group_best != 1 && d->group_best != 2) return fail(B200SEQ_ERR_INVALID_ARG, "%s: a group's score is its largest (1) or the sum of its two largest (2)", what);
+    if (d->kind == 2 && !d->renorm) return fail(B200SEQ_ERR_INVALID_ARG, "%s: weights over the chosen logits are always normalised", what);
+    if (d->groups > 1 && (d->E % d->groups || d->keep < 1 || d->keep > d->groups || (int64_t)d->keep * (d->E / d->groups) < d->top))
+        return fail(B200SEQ_ERR_INVALID_ARG, "%s: groups must divide the experts and the kept groups must hold `top` experts", what);
+    const bool grouped = d->groups > 1;
+    r = RouteRule{d->E, grouped ? d->groups : 1, grouped ? d->keep : 1, d->top, d->kind, d->correction, d->group_best, d->renorm, d->scale};
+    return 0;
+}
+
+int b200seq_moe_route_rule(const float* z, int64_t ldz, int T, const b200seq_route_desc* d, int32_t* ids, float* wts, int32_t* counts, void* stream) {
+    RouteRule rule;
+    if (int rc = route_rule(d, rule, "moe_route")) return rc;
+    const int E = d->E, top = d->top;
     if (!z || !ids || !wts || T < 0 || E < 1 || E > MOE_MAX_E || top < 1 || top > E || ldz < E) return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: bad arguments (experts <= %d)", MOE_MAX_E);
-    if (groups > 1 && (E % groups || keep < 1 || keep > groups || (int64_t)keep * (E / groups) < top))
-        return fail(B200SEQ_ERR_INVALID_ARG, "moe_route: groups must divide the experts and the kept groups must hold `top` experts");
     cudaStream_t cs = (cudaStream_t)stream;
     if (counts) {
         cudaError_t e = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int32_t), cs);
         if (e != cudaSuccess) return cuda_status(e, "moe_route memset");
     }
     if (T == 0) return 0;
-    const int g = groups > 1 ? groups : 1;
-    moe_route_kernel<<<T, 32, (size_t)(2 * E + g) * sizeof(float), cs>>>(z, ldz, E, g, groups > 1 ? keep : 1, top, ids, wts, counts, kind, correction);
+    moe_route_kernel<<<T, 32, (size_t)(2 * E + rule.groups) * sizeof(float), cs>>>(z, ldz, rule, ids, wts, counts);
     SEQ_LAUNCH_CHECK("moe_route");
     return 0;
 }
@@ -570,25 +595,30 @@ int b200seq_moe_router(const void* x, int x_dtype, int64_t ldx_, const void* w, 
 
 int b200seq_moe_router_ex(const void* x, int x_dtype, int64_t ldx_, const void* w, int T, int NR, int K, int E, int groups, int keep, int top, int kind,
                           const float* correction, float* z, int64_t ldz, int32_t* ids, float* wts, void* stream) {
-    if (kind < 0 || kind > 2) return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: score kind 0 (sigmoid), 1 (soft-max) or 2 (soft-max over the chosen)");
+    const b200seq_route_desc d{E, groups, keep, top, kind, 2, 1, 1.f, correction};
+    return b200seq_moe_router_rule(x, x_dtype, ldx_, w, T, NR, K, &d, z, ldz, ids, wts, stream);
+}
+
+int b200seq_moe_router_rule(const void* x, int x_dtype, int64_t ldx_, const void* w, int T, int NR, int K, const b200seq_route_desc* d, float* z, int64_t ldz,
+                            int32_t* ids, float* wts, void* stream) {
+    RouteRule rule;
+    if (int rc = route_rule(d, rule, "moe_router")) return rc;
+    const int E = d->E, top = d->top;
     if (!x || !w || !z || !ids || !wts || T < 0 || T > 8 || E < 1 || E > MOE_MAX_E || NR < E || K < 1 || ldx_ < K || ldz < NR || top < 1 || top > E)
         return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: bad arguments (at most 8 tokens, experts <= %d)", MOE_MAX_E);
-    if (groups > 1 && (E % groups || keep < 1 || keep > groups || (int64_t)keep * (E / groups) < top))
-        return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: groups must divide the experts and the kept groups must hold `top` experts");
     if (x_dtype != B200SEQ_F32 && x_dtype != B200SEQ_BF16) return fail(B200SEQ_ERR_INVALID_ARG, "moe_router: activation dtype");
     if (T == 0) return 0;
-    const int g = groups > 1 ? groups : 1, kp = groups > 1 ? keep : 1;
-    const size_t smem = (size_t)(NR + 2 * E + g) * sizeof(float);
+    const size_t smem = (size_t)(NR + 2 * E + rule.groups) * sizeof(float);
     const size_t es = x_dtype == B200SEQ_F32 ? 4 : 2;
     const bool vec = K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (ldx_ * es) % 16 == 0;
     cudaStream_t cs = (cudaStream_t)stream;
     const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
     if (x_dtype == B200SEQ_F32) {
-        if (vec) moe_router_rows_kernel<float, true><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, E, g, kp, top, ids, wts, kind, correction);
-        else moe_router_rows_kernel<float, false><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, E, g, kp, top, ids, wts, kind, correction);
+        if (vec) moe_router_rows_kernel<float, true><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
+        else moe_router_rows_kernel<float, false><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
     } else {
-        if (vec) moe_router_rows_kernel<__nv_bfloat16, true><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, E, g, kp, top, ids, wts, kind, correction);
-        else moe_router_rows_kernel<__nv_bfloat16, false><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, E, g, kp, top, ids, wts, kind, correction);
+        if (vec) moe_router_rows_kernel<__nv_bfloat16, true><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
+        else moe_router_rows_kernel<__nv_bfloat16, false><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
     }
     SEQ_LAUNCH_CHECK("moe_router");
     return 0;

@@ -13,6 +13,8 @@
 //   B        start_c = S;  S = d^L S + U_c   in chunk order per entry; the last S goes to the sequence's slot
 //   C        o_i = d^(i+1) start_c^T q_i + sum_(j<=i) d^(i-j) (q_i . k_j) v_j
 //   finish   unit norm over V and gate, written in the activation type
+// One norm over all heads of a token (norm_w): its division is deferred past the output projection, which is linear in it.  Pass C (and the decode
+// kernel, then one per entry, head and tile of value columns) writes o * weight * gate and the tile's sum of squares; no finish pass.
 // Powers of the decay are exp2(n * log2 d) with log2 d handed in (computed in double by the caller).
 #include "seq_common.cuh"
 
@@ -21,6 +23,7 @@ namespace b200seq {
 constexpr int RET_C = 64;    // tokens per chunk
 constexpr int RET_DS = 32;   // key dimensions per staged slab
 constexpr int RET_NT = 256;
+constexpr int RET_SV = 32;   // value columns per block of the tiled decode kernel
 
 // ---- rotary positions on head vectors inside projection rows ------------------------------------------------------------------------
 // grid (T), any block size: heads [nheads][D] at column `col` of row t; the first rot_dims dimensions of every head turn by
@@ -69,25 +72,18 @@ struct RetArgs {
     float* o_raw;       // [T][H * V]
     void* out;
     int out_dtype;
+    const float* norm_w;   // [H * V]: one deferred norm over all heads; null: a unit norm per head
+    int gate_sigmoid;
+    float* sumsq;          // [T][partials]
 };
+__device__ __forceinline__ float ret_gate(const RetArgs& a, float g) { return a.gate_sigmoid ? sigmoidf_acc(g) : siluf_acc(g); }
 
-// ---- decode: grid (B, H), RET_NT threads ------------------------------------------------------------------------------------------------
-// dynamic shared memory: q [D] | k [D] | partial o [4][V] | 40 floats of reduction scratch
-__global__ void __launch_bounds__(RET_NT) retention_step_kernel(const RetArgs a, const b200seq_step st) {
-    extern __shared__ __align__(16) float sm[];
-    const int D = a.D, V = a.V, H = a.H;
-    float* qs = sm;
-    float* ks = qs + D;
-    float* part = ks + D;        // [4][V]
-    float* red = part + 4 * V;
-    const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
-    const int t = st.ent_start[e];
-    const float pos = (float)st.tok_pos[t];
-    const float* row = a.proj + (int64_t)t * a.ld;
-    const float* qg = row + a.q_col + (int64_t)h * D;
-    const float* kg = row + a.k_col + (int64_t)h * D;
+// q and k of one head (rotated, k scaled) to shared memory
+__device__ __forceinline__ void ret_load_qk(const RetArgs& a, const float* row, int h, float pos, float* qs, float* ks) {
+    const float* qg = row + a.q_col + (int64_t)h * a.D;
+    const float* kg = row + a.k_col + (int64_t)h * a.D;
     const int np = a.rot_dims >> 1;
-    for (int i = tid; i < D; i += RET_NT) {
+    for (int i = threadIdx.x; i < a.D; i += RET_NT) {
         float q = qg[i], k = kg[i];
         if (i < a.rot_dims) {
             const int pi = a.rot_half ? (i < np ? i : i - np) : (i >> 1);
@@ -102,6 +98,83 @@ __global__ void __launch_bounds__(RET_NT) retention_step_kernel(const RetArgs a,
         }
         qs[i] = q, ks[i] = k * a.k_scale;
     }
+}
+
+// ---- decode, one norm over all heads: grid (B, H, tiles of RET_SV value columns), RET_NT threads -------------------------------------------------
+// thread = (value column, one of 8 groups of key dimensions); EPT: state elements a thread keeps in registers (D <= 8 * EPT), requested before anything is
+// waited for; 0: any D.  dynamic shared memory: q [D] | k [D] | partial o [8][RET_SV]
+template <int EPT>
+__global__ void __launch_bounds__(RET_NT) retention_step_tile_kernel(const RetArgs a, const b200seq_step st) {
+    extern __shared__ __align__(16) float sm[];
+    const int D = a.D, V = a.V, H = a.H;
+    float *qs = sm, *ks = qs + D, *part = ks + D;
+    const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vt = tid & (RET_SV - 1), dg = tid / RET_SV;
+    const int v = blockIdx.z * RET_SV + vt;
+    const bool in = v < V;
+    const int t = st.ent_start[e];
+    float* S = a.state + ((int64_t)st.ent_slot[e] * H + h) * D * V + v;
+    const bool fresh = st.ent_pos0[e] == 0;
+    constexpr int NE = EPT > 0 ? EPT : 1;
+    float s[NE];
+    if (EPT > 0) {
+#pragma unroll
+        for (int j = 0; j < NE; ++j) {
+            const int d = dg + 8 * j;
+            s[j] = (!fresh && in && d < D) ? S[(int64_t)d * V] : 0.f;
+        }
+    }
+    const float* row = a.proj + (int64_t)t * a.ld;
+    const float vv = in ? row[a.v_col + (int64_t)h * V + v] : 0.f;
+    const float dec = a.decay[h];
+    ret_load_qk(a, row, h, (float)st.tok_pos[t], qs, ks);
+    __syncthreads();
+    float o = 0.f;
+    if (in) {
+        if (EPT > 0) {
+#pragma unroll
+            for (int j = 0; j < NE; ++j) {
+                const int d = dg + 8 * j;
+                if (d < D) {
+                    s[j] = fmaf(dec, s[j], ks[d] * vv);
+                    S[(int64_t)d * V] = s[j];
+                    o = fmaf(s[j], qs[d], o);
+                }
+            }
+        } else {
+            for (int d = dg; d < D; d += 8) {
+                const float n = fmaf(dec, fresh ? 0.f : S[(int64_t)d * V], ks[d] * vv);
+                S[(int64_t)d * V] = n;
+                o = fmaf(n, qs[d], o);
+            }
+        }
+    }
+    part[dg * RET_SV + vt] = o;
+    __syncthreads();
+    if (dg == 0) {
+        o = 0.f;
+#pragma unroll
+        for (int g = 0; g < 8; ++g) o += part[g * RET_SV + vt];
+        const float ss = warp_sum(o * o);
+        const int c = h * V + v;
+        if (in) store_act(a.out, a.out_dtype, (int64_t)t * H * V + c, o * a.norm_w[c] * ret_gate(a, row[a.g_col + c]));
+        if (vt == 0) a.sumsq[((int64_t)t * H + h) * gridDim.z + blockIdx.z] = ss;
+    }
+}
+
+// ---- decode: grid (B, H), RET_NT threads ------------------------------------------------------------------------------------------------
+// dynamic shared memory: q [D] | k [D] | partial o [4][V] | 40 floats of reduction scratch
+__global__ void __launch_bounds__(RET_NT) retention_step_kernel(const RetArgs a, const b200seq_step st) {
+    extern __shared__ __align__(16) float sm[];
+    const int D = a.D, V = a.V, H = a.H;
+    float* qs = sm;
+    float* ks = qs + D;
+    float* part = ks + D;        // [4][V]
+    float* red = part + 4 * V;
+    const int e = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int t = st.ent_start[e];
+    const float pos = (float)st.tok_pos[t];
+    const float* row = a.proj + (int64_t)t * a.ld;
+    ret_load_qk(a, row, h, pos, qs, ks);
     __syncthreads();
     const float dec = a.decay[h];
     float* S = a.state + ((int64_t)st.ent_slot[e] * H + h) * D * V;
@@ -133,7 +206,7 @@ __global__ void __launch_bounds__(RET_NT) retention_step_kernel(const RetArgs a,
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)V + a.eps);
     const float* gg = row + a.g_col + (int64_t)h * V;
-    for (int v = tid; v < V; v += RET_NT) store_act(a.out, a.out_dtype, ((int64_t)t * H + h) * V + v, part[v] * rinv * siluf_acc(gg[v]));
+    for (int v = tid; v < V; v += RET_NT) store_act(a.out, a.out_dtype, ((int64_t)t * H + h) * V + v, part[v] * rinv * ret_gate(a, gg[v]));
 }
 
 // ---- chunked form -------------------------------------------------------------------------------------------------------------------------
@@ -322,6 +395,37 @@ __global__ void __launch_bounds__(RET_NT) retention_out_kernel(const RetArgs a, 
             }
         }
     }
+    if (a.norm_w) {   // weight and gate here; the tile's sum of squares for the norm over all heads
+        const int vb = v0 + tx * 4;
+        const bool v4 = (V & 3) == 0;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int qi = ty * 4 + i;
+            const bool row_in = qi < len;
+            const int64_t t = row0 + qi;
+            const float w = pw[qi + 1];
+            float o[4], ss = 0.f;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                o[u] = (row_in && vb + u < V) ? fmaf(w, acs[i][u], acc[i][u]) : 0.f;
+                ss = fmaf(o[u], o[u], ss);
+            }
+#pragma unroll
+            for (int m = 8; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);   // the 16 lanes of a row
+            if (!row_in) continue;
+            if (tx == 0) a.sumsq[(t * H + h) * gridDim.x + blockIdx.x] = ss;
+            if (vb >= V) continue;
+            const int64_t ob = (t * H + h) * V + vb;
+            const float* gg = a.proj + t * a.ld + a.g_col + (int64_t)h * V + vb;
+            const float* nw = a.norm_w + (int64_t)h * V + vb;
+            if (v4) {
+                store_act4(a.out, a.out_dtype, ob, make_float4(o[0] * nw[0] * ret_gate(a, gg[0]), o[1] * nw[1] * ret_gate(a, gg[1]), o[2] * nw[2] * ret_gate(a, gg[2]), o[3] * nw[3] * ret_gate(a, gg[3])));
+            } else {
+                for (int u = 0; u < 4 && vb + u < V; ++u) store_act(a.out, a.out_dtype, ob + u, o[u] * nw[u] * ret_gate(a, gg[u]));
+            }
+        }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int qi = ty * 4 + i;
@@ -345,7 +449,7 @@ __global__ void retention_finish_kernel(const RetArgs a) {
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)V + a.eps);
     const float* gg = a.proj + (int64_t)t * a.ld + a.g_col + (int64_t)h * V;
-    for (int v = threadIdx.x; v < V; v += blockDim.x) store_act(a.out, a.out_dtype, ((int64_t)t * a.H + h) * V + v, o[v] * rinv * siluf_acc(gg[v]));
+    for (int v = threadIdx.x; v < V; v += blockDim.x) store_act(a.out, a.out_dtype, ((int64_t)t * a.H + h) * V + v, o[v] * rinv * ret_gate(a, gg[v]));
 }
 
 }  // namespace b200seq
@@ -363,6 +467,8 @@ extern "C" int b200seq_rotary(float* x, int64_t ld, int col, int nheads, int D, 
     return 0;
 }
 
+extern "C" int b200seq_retention_partials(int T, int B, int H, int V) { return H * (T == B ? (V + RET_SV - 1) / RET_SV : (V + 63) / 64); }
+
 extern "C" size_t b200seq_retention_scratch_floats(int T, int B, int H, int D, int V) {
     if (T < 1 || B < 1 || T == B) return 0;
     const size_t chunks = (size_t)(T + RET_C - 1) / RET_C + (size_t)B;
@@ -376,14 +482,25 @@ extern "C" int b200seq_retention(float* proj, int64_t ld, const b200seq_step* st
     if (d->rot_dims < 0 || d->rot_dims > d->D || (d->rot_dims & 1) || (d->rot_dims > 0 && !d->rot_freq))
         return fail(B200SEQ_ERR_INVALID_ARG, "retention: rotary dimensions must be even, at most the key size, with a frequency table");
     if (out_dtype != B200SEQ_F32 && out_dtype != B200SEQ_BF16) return fail(B200SEQ_ERR_INVALID_ARG, "retention: output dtype");
+    if (d->norm_w && !d->sumsq) return fail(B200SEQ_ERR_INVALID_ARG, "retention: a norm over all heads needs a place for the sums of squares");
     if (st->T == 0 || st->B == 0) return 0;
     cudaStream_t cs = (cudaStream_t)stream;
     RetArgs a{proj, ld, d->q_col, d->k_col, d->v_col, d->g_col, d->H, d->D, d->V, d->decay, d->eps, d->rot_dims, d->rot_half, d->rot_freq, d->rot_scale, d->k_scale,
-              state, nullptr, nullptr, out, out_dtype};
+              state, nullptr, nullptr, out, out_dtype, d->norm_w, d->gate_sigmoid, d->sumsq};
     if (st->T == st->B) {
         const size_t smem = ((size_t)2 * d->D + 4 * d->V + 40) * sizeof(float);
         if (smem > 48 * 1024) return fail(B200SEQ_ERR_UNSUPPORTED, "retention: head sizes too large");
         if (st->B > 65535 || d->H > 65535) return fail(B200SEQ_ERR_UNSUPPORTED, "retention: too many entries or heads");
+        if (d->norm_w) {
+            const size_t tile = ((size_t)2 * d->D + 8 * RET_SV) * sizeof(float);
+            const dim3 grid(st->B, d->H, (d->V + RET_SV - 1) / RET_SV);
+            if (d->D <= 64) retention_step_tile_kernel<8><<<grid, RET_NT, tile, cs>>>(a, *st);
+            else if (d->D <= 128) retention_step_tile_kernel<16><<<grid, RET_NT, tile, cs>>>(a, *st);
+            else if (d->D <= 256) retention_step_tile_kernel<32><<<grid, RET_NT, tile, cs>>>(a, *st);
+            else retention_step_tile_kernel<0><<<grid, RET_NT, tile, cs>>>(a, *st);
+            SEQ_LAUNCH_CHECK("retention step");
+            return 0;
+        }
         retention_step_kernel<<<dim3(st->B, d->H), RET_NT, smem, cs>>>(a, *st);
         SEQ_LAUNCH_CHECK("retention step");
         return 0;
@@ -404,6 +521,7 @@ extern "C" int b200seq_retention(float* proj, int64_t ld, const b200seq_step* st
     SEQ_LAUNCH_CHECK("retention combine pass");
     retention_out_kernel<<<dim3(vt, chunks, d->H), RET_NT, 0, cs>>>(a, *st);
     SEQ_LAUNCH_CHECK("retention output pass");
+    if (d->norm_w) return 0;
     retention_finish_kernel<<<dim3(st->T, d->H), d->V <= 64 ? 64 : 128, 0, cs>>>(a);
     SEQ_LAUNCH_CHECK("retention finish");
     return 0;

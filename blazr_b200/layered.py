@@ -14,7 +14,9 @@ wrapped in the pieces a design switches on.  These layouts of the residual path 
              may pass a soft cap (blazr_b200/pafelorn.py);
   "sandwich": sublayers in sequence, each normed on both sides, x <- x + norm(sublayer(norm(x))); positions may enter as a sinusoid at the
              embedding, every layer may add a gated, projected row of a per-token table, and a span of layers may run several times with
-             rows added in front of each pass (blazr_b200/vodelix.py).
+             rows added in front of each pass (blazr_b200/vodelix.py);
+  "parallel": mixer and feed-forward read the same RMS-normed input, x <- x + m (mixer(h) + ff(h)); a mixer may be two branches side by side
+             (an attention beside a selective scan); a span of layers may run several times (blazr_b200/zetunex.py).
 The mechanisms are parameterised (window / chunk / pooled-block size, score scale, unit-norm epsilon, rotary table, gate, state
 size, activation kind, router groups, ...) so that another design can list them in another combination; a design is a function
 config.json -> LayeredConfig.
@@ -120,12 +122,17 @@ class SsmSpec:
 @dataclass
 class RetentionSpec:
     """linear attention with one fixed decay per head, no soft-max and no denominator: S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t;
-    rotary positions on q and k, k times dim^(-1/2), every head's o divided by its root mean square, times silu(gate), then the output projection"""
+    rotary positions on q and k, k times key_scale, then norm "head": every head's o divided by its root mean square, or "joint": one weighted RMS norm
+    over all heads (tensor "mix.norm"; layout "parallel"); times gate(g) ("silu" or "sigmoid"), then the output projection"""
     heads: int
     dim: int                 # per-head query / key size
     vdim: int                # per-head value size
     decay: List[float] = field(default_factory=list)
     rot: Optional[RotarySpec] = None
+    key_scale: Optional[float] = None   # None: dim^(-1/2)
+    qkv_silu: bool = False              # q, k and v pass silu (layout "parallel")
+    norm: str = "head"
+    gate: str = "silu"
 
 
 @dataclass
@@ -165,6 +172,17 @@ class RgLruSpec:
 
 
 @dataclass
+class ScanSpec:
+    """selective scan: W_in h = [x | z] (inner each), x <- silu(causal_conv(x)), W_x x = [low (dt_rank) | B (state) | C (state)], dt = softplus(W_dt low + b),
+    S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n, y_c = sum_n S[c, n] C_n + D_c x_c; output W_o (y * silu(z)); f32 state and the last
+    conv - 1 convolution inputs per sequence"""
+    inner: int
+    state: int
+    conv: int
+    dt_rank: int
+
+
+@dataclass
 class DeltaSpec:
     """delta-rule recurrence with a decay and a removal rate per head and key channel: with the unit key u = k / sqrt(sum k^2 + unit_eps),
     S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T, o_t = S_t^T r; w = exp(-decay_scale sigmoid(W_2 tanh(W_1 h) + w0)), a = sigmoid(W_a h + b);
@@ -181,7 +199,7 @@ class TwoBranchSpec:
     """an attention (left) and a recurrence (right) read the same input; result = left_scale * left + right_scale * right, each branch first
     RMS-normed over the model width with a weight of its own when branch_norm"""
     left: AttentionSpec
-    right: object            # MinGruSpec | RgLruSpec
+    right: object            # MinGruSpec | RgLruSpec (layout "out_norm"), ScanSpec (layout "parallel")
     left_scale: float = 1.0
     right_scale: float = 1.0
     branch_norm: bool = False
@@ -222,6 +240,10 @@ class MoeFfSpec:
     alpha: float = 1.702
     up_shift: float = 1.0
     shared_limit: float = 0.0
+    # ---- learned routers -------------------------------------------------------------------------------------------------------------------------------
+    group_best: int = 2      # a group's score: the sum of its two largest scores, or (1) its largest
+    renorm: bool = True      # weights divided by the sum of the chosen ones
+    route_scale: float = 1.0 # weights times this
 
 
 @dataclass
@@ -229,9 +251,9 @@ class LayerSpec:
     kind: str                # "attention" | "ssm" | "retention" | "latent_attention" | "two_branch" | "delta"
     mixer: object
     ff: Optional[object]     # DenseFfSpec | MoeFfSpec | None
-    weights_of: Optional[int] = None   # layouts "post", "sandwich": the layer has no tensors of its own and uses those of this (earlier) layer, with its own cache / state
-    tensors: Optional[int] = None      # layout "sandwich": the number in the layer's tensor names when it is not its place in the list (layers that run several times)
-    enter: Optional[tuple] = None      # layout "sandwich": added to x in front of this layer: (the embedding output too?, row of "loop.step" or None)
+    weights_of: Optional[int] = None   # layouts "post", "sandwich", "parallel": the layer has no tensors of its own and uses those of this (earlier) layer, with its own cache / state
+    tensors: Optional[int] = None      # layouts "sandwich", "parallel": the number in the layer's tensor names when it is not its place in the list (layers that run several times)
+    enter: Optional[tuple] = None      # layouts "sandwich", "parallel": added to x in front of this layer: (the embedding output too?, row of "loop.step" or None)
 
 
 @dataclass
@@ -245,7 +267,7 @@ class LayeredConfig:
     canon_taps: int          # taps of the convolution in front of every sublayer
     embed_scale: float
     layers: List[LayerSpec] = field(default_factory=list)
-    layout: str = "streams"  # "streams" | "depth" (see the module text)
+    layout: str = "streams"  # see the module text
     tied_head: bool = True   # the output projection is the embedding table; False: a tensor "head"
     depth_average: bool = True   # layout "depth": layer i has weights "l<i>.dwa" [i + 2] over the embedding and the results of layers 0..i
     post_alpha: float = 1.0      # layout "post": weight of the residual in the sum that is normed
@@ -253,7 +275,19 @@ class LayeredConfig:
     logit_softcap: float = 0.0       # > 0: logits <- cap * tanh(logits / cap)
     norm_shift: float = 0.0          # layout "sandwich": the layer norms' stored weights plus this are what multiplies
     position_base: float = 0.0       # layout "sandwich": > 0: sin / cos(position * base^(-2i / width)) is added to entries 2i / 2i + 1 of the embedding
+    residual_mult: float = 1.0       # layout "parallel": what the sublayers' results are multiplied by
     token_side: int = 0              # layout "sandwich": > 0: every layer adds a row of this size of the table "side.embed", gated and projected
+
+
+def loop_runs(n: int, start: int = 0, stop: int = 0, times: int = 0) -> list:
+    """n layers of which start .. stop - 1 run `times` times in a row (times 0: no loop): (layer, pass or None outside the loop, first layer of its pass) in
+    the order they run"""
+    if not times:
+        return [(i, None, False) for i in range(n)]
+    runs = [(i, None, False) for i in range(start)]
+    for t in range(times):
+        runs += [(i, t, i == start) for i in range(start, stop)]
+    return runs + [(i, None, False) for i in range(stop, n)]
 
 
 class _Rows:
@@ -335,6 +369,18 @@ class _Workspace:
             self.side_g = torch.empty((cap, max(1, cfg.token_side)), **act)
             self.ff_inner = torch.empty((cap, max(1, model.max_ff_inner)), **act)
             self.ff_proj = torch.empty((cap, max(1, model.max_ff_proj)), **f32)
+        if cfg.layout == "parallel":    # second branch, the scan's intermediates and work area (it runs beside the attention), sums of squares, the feed-forward's own buffers
+            self.y2 = torch.empty((cap, W), **f32)
+            self.y3 = torch.empty((cap, W), **f32)
+            self.inner_b = torch.empty((cap, max(1, model.max_rinner)), **act)
+            self.conv_a = torch.empty((cap, max(1, model.max_rinner)), **act)
+            self.dbc = torch.empty((cap, max(1, model.max_dbc)), **f32)
+            self.low = torch.empty((cap, max(1, model.max_rank)), **act)
+            self.dtz = torch.empty((cap, max(1, model.max_rinner)), **f32)
+            self.sumsq = torch.empty((cap, max(1, model.max_sumsq)), **f32)
+            self.scratch_b = torch.empty(max(1, model.scan_scratch_floats(cap)), **f32)
+            self.ff_inner = torch.empty((cap, max(1, model.max_ff_inner)), **act)
+            self.ff_proj = torch.empty((cap, max(1, model.max_ff_proj)), **f32)
         mo = model.moe_dims
         if mo is not None:              # mixture of experts: router logits, choices, sort, per-pair intermediates
             E1, top, F = mo
@@ -408,13 +454,15 @@ class LayeredModel:
         def hc(pre):    # (in [S], post = out [S] | mix [S, S])
             return vec(pre + "in"), torch.cat([get(pre + "out").float().reshape(-1), get(pre + "mix").float().reshape(-1)]).contiguous().to(dev)
 
-        if cfg.layout not in ("streams", "depth", "post", "out_norm", "sandwich"):
+        if cfg.layout not in ("streams", "depth", "post", "out_norm", "sandwich", "parallel"):
             raise ValueError(f"unknown residual layout {cfg.layout}")
-        depth, post, outn, sandwich = (cfg.layout == l for l in ("depth", "post", "out_norm", "sandwich"))
+        depth, post, outn, sandwich, parallel = (cfg.layout == l for l in ("depth", "post", "out_norm", "sandwich", "parallel"))
         if cfg.layout != "streams" and (S != 1 or cfg.canon_taps > 1):
             raise ValueError("only the layout of several streams has more than one residual stream and carried convolutions")
         if not sandwich and (cfg.norm_shift or cfg.position_base or cfg.token_side):
             raise ValueError("shifted norm weights, sinusoidal positions and the token-dependent addition are wired into the sandwich layout")
+        if not parallel and cfg.residual_mult != 1.0:
+            raise ValueError("a multiplier on the sublayers' results is wired into the parallel layout")
         self.embed = lin("embed")
         self.head = self.embed if cfg.tied_head else lin("head")
         self.final_norm = vec("final.norm") + cfg.norm_shift
@@ -439,7 +487,8 @@ class LayeredModel:
             raise ValueError("loop.step has one row of the model width per pass")
         self.max_rank = self.max_wz = 1      # sandwich layout: low-rank decay branch (its rank, its output width)
         self.layers: List[Dict[str, object]] = []
-        self.max_rinner = 1      # out_norm layout: widest recurrent branch
+        self.max_rinner = 1      # out_norm, parallel layouts: widest recurrent branch
+        self.max_dbc = self.max_sumsq = 1    # parallel layout: widest scan projection, most sums of squares of a joint head norm
         self.max_proj = self.max_xbc = self.max_inner = 1
         self.max_ff_inner = self.max_ff_proj = 1      # depth layout: sizes of the feed-forward branch's own intermediates
         self.moe_dims = None      # (experts + 1, top, expert ff): largest over the layers
@@ -456,6 +505,9 @@ class LayeredModel:
                 continue
             if sandwich:
                 self.layers.append(self._sandwich_layer(i, ls, lin, vec, get))
+                continue
+            if parallel:
+                self.layers.append(self._parallel_layer(i, ls, lin, vec, get))
                 continue
             L: Dict[str, object] = {"spec": ls}
             p = f"l{i}."
@@ -514,6 +566,7 @@ class LayeredModel:
                 L["norm2"] = vec(p + "norm2")
                 router = [p + "mlp.router"] + ([p + "mlp.shared.sg"] if f.shared_ff and f.shared_gate else [])
                 L["w_router"] = lin(*router)          # the shared expert's token gate rides as one more row
+                L["route"] = seqops.route_desc(f.experts, f.groups, f.keep, f.top, seqops.ROUTE_SIGMOID, group_best=f.group_best, renorm=f.renorm, scale=f.route_scale)
                 L["w_eup"] = torch.stack([lin(p + f"mlp.e{e}.up") for e in range(f.experts)]).contiguous()
                 L["w_edown"] = torch.stack([lin(p + f"mlp.e{e}.down") for e in range(f.experts)]).contiguous()
                 if tuple(L["w_router"].shape) != (len(router) - 1 + f.experts, W) or tuple(L["w_eup"].shape[1:]) != (f.ff, W) or tuple(L["w_edown"].shape[1:]) != (W, f.ff):
@@ -595,20 +648,9 @@ class LayeredModel:
             return torch.from_numpy(fr).to(dev), scale
 
         if ls.kind == "retention":
-            import math
-            H, D, V = m.heads, m.dim, m.vdim
-            L["w_in"] = lin(p + "mix.q", p + "mix.k", p + "mix.v", p + "mix.g")
-            L["w_o"] = lin(p + "mix.o")
-            if tuple(L["w_in"].shape) != (2 * H * D + 2 * H * V, W) or tuple(L["w_o"].shape) != (W, H * V) or len(m.decay) != H:
-                raise ValueError(f"layer {i}: retention tensor shapes / decay list do not fit the configuration")
-            if any(not 0.0 < float(d) <= 1.0 for d in m.decay):
-                raise ValueError(f"layer {i}: decays lie in (0, 1]")
-            L["decay"] = torch.tensor([[float(d) for d in m.decay], [math.log2(float(d)) for d in m.decay]], dtype=torch.float64).to(torch.float32).to(dev)
-            L["rot_freq"], rot_scale = rotary(m.rot, D, "the key size")
-            if m.rot is not None and m.rot.layout not in ("half", "interleaved"):
-                raise ValueError(f"layer {i}: unknown rotary layout {m.rot.layout}")
-            L["desc"] = seqops.retention_desc(H, D, V, L["decay"], cfg.eps, float(D) ** -0.5, rot_freq=L["rot_freq"],
-                                              rot_half=m.rot is not None and m.rot.layout == "half", rot_scale=rot_scale)
+            if m.qkv_silu or m.norm != "head":
+                raise ValueError(f"layer {i}: silu on q, k, v and a norm over all heads are wired into the parallel layout")
+            self._retention_weights(L, i, m, p + "mix.", lin, vec)
         elif ls.kind == "latent_attention":
             H, Dn, Rd, V, R, Rq = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.q_rank
             if m.rot is not None and (m.rot.dims != Rd or m.rot.layout != "interleaved"):
@@ -653,6 +695,30 @@ class LayeredModel:
             self.weight_bytes += (L["w_gu"].numel() + L["w_down"].numel()) * 2
         self._post_sizes(L, ls)
         return L
+
+    def _retention_weights(self, L, i: int, m: RetentionSpec, ap: str, lin, vec) -> None:
+        import math
+        H, D, V, W, dev = m.heads, m.dim, m.vdim, self.cfg.width, self.dev
+        L["w_in"] = lin(ap + "q", ap + "k", ap + "v", ap + "g")
+        L["w_o"] = lin(ap + "o")
+        if tuple(L["w_in"].shape) != (2 * H * D + 2 * H * V, W) or tuple(L["w_o"].shape) != (W, H * V) or len(m.decay) != H:
+            raise ValueError(f"layer {i}: retention tensor shapes / decay list do not fit the configuration")
+        if any(not 0.0 < float(d) <= 1.0 for d in m.decay):
+            raise ValueError(f"layer {i}: decays lie in (0, 1]")
+        if m.norm not in ("head", "joint") or m.gate not in ("silu", "sigmoid"):
+            raise ValueError(f"layer {i}: unknown head norm {m.norm} / gate {m.gate}")
+        L["decay"] = torch.tensor([[float(d) for d in m.decay], [math.log2(float(d)) for d in m.decay]], dtype=torch.float64).to(torch.float32).to(dev)
+        L["rot_freq"], rot_scale = None, 1.0
+        if m.rot is not None:
+            if m.rot.dims < 2 or m.rot.dims % 2 or m.rot.dims > D or m.rot.layout not in ("half", "interleaved"):
+                raise ValueError(f"layer {i}: rotary dimensions must be even and at most the key size, layout half or interleaved")
+            fr, rot_scale = m.rot.table()
+            L["rot_freq"] = torch.from_numpy(fr).to(dev)
+        L["mnorm"] = vec(ap + "norm") if m.norm == "joint" else None
+        if L["mnorm"] is not None and L["mnorm"].numel() != H * V:
+            raise ValueError(f"layer {i}: the norm over all heads has one weight per value")
+        L["desc"] = seqops.retention_desc(H, D, V, L["decay"], self.cfg.eps, float(D) ** -0.5 if m.key_scale is None else float(m.key_scale), rot_freq=L["rot_freq"],
+                                          rot_half=m.rot is not None and m.rot.layout == "half", rot_scale=rot_scale, norm_w=L["mnorm"], gate_sigmoid=m.gate == "sigmoid")
 
     # ---- layout "out_norm": weights of one layer ------------------------------------------------------------------------------------------
     def _out_layer(self, i: int, ls: "LayerSpec", lin, vec, get) -> Dict[str, object]:
@@ -877,6 +943,91 @@ class LayeredModel:
             self.weight_bytes += (L["side_gate"].numel() + L["side_proj"].numel()) * 2
         return L
 
+    # ---- layout "parallel": weights of one layer ----------------------------------------------------------------------------------------------
+    def _parallel_layer(self, i: int, ls: "LayerSpec", lin, vec, get) -> Dict[str, object]:
+        """a layer that runs again (weights_of) shares every tensor with its first run and gets a cache / state of its own in allocate()"""
+        cfg, dev, W = self.cfg, self.dev, self.cfg.width
+        m, f = ls.mixer, ls.ff
+        n = i if ls.tensors is None else ls.tensors
+        if ls.enter is not None and ls.enter[0]:
+            raise ValueError(f"layer {i}: the embedding output in front of a pass is wired into the sandwich layout")
+        if ls.weights_of is not None:
+            j = ls.weights_of
+            if not 0 <= j < i or cfg.layers[j].weights_of is not None:
+                raise ValueError(f"layer {i}: weights_of must name an earlier layer that has tensors of its own")
+            if cfg.layers[j].kind != ls.kind or cfg.layers[j].mixer != m or cfg.layers[j].ff != f:
+                raise ValueError(f"layer {i}: a layer that shares weights has the sizes of the layer it shares them with")
+            return dict(self.layers[j], spec=ls)
+        L: Dict[str, object] = {"spec": ls, "silu": (0, 0)}
+        p = f"l{n}."
+        L["norm1"] = vec(p + "norm1")
+        if L["norm1"].numel() != W:
+            raise ValueError(f"layer {i}: norm weight does not fit the width")
+        if ls.kind == "retention":
+            self._retention_weights(L, i, m, p + "mix.", lin, vec)
+            H, D, V = m.heads, m.dim, m.vdim
+            if m.qkv_silu:
+                L["silu"] = (0, 2 * H * D + H * V)
+            self.weight_bytes += (L["w_in"].numel() + L["w_o"].numel()) * 2
+            self.max_inner = max(self.max_inner, H * V)
+            if m.norm == "joint":
+                self.max_sumsq = max(self.max_sumsq, seqops.retention_partials(1, 1, H, V), seqops.retention_partials(2, 1, H, V))
+        elif ls.kind in ("attention", "two_branch"):
+            att, right, ap = (m, None, p + "mix.") if ls.kind == "attention" else (m.left, m.right, p + "mix.left.")
+            if att.diff is not None or att.kv_from is not None or att.out_bias:
+                raise ValueError(f"layer {i}: differential attention, another layer's keys and an output bias are not wired into the parallel layout")
+            rows = _Rows(i, get, W)
+            self._attention_rows(i, att, ap, rows)
+            n_att = rows.width
+            if right is not None:
+                if not isinstance(right, ScanSpec):
+                    raise ValueError(f"layer {i}: recurrent branch {type(right).__name__} is not wired into the parallel layout")
+                rows.add(p + "mix.right.in", 2 * right.inner)
+            L["w_in"], L["in_bias"] = rows.stacked(dev)
+            self._attention_rest(L, i, att, ap, n_att, lin, vec, get)
+            if right is not None:
+                self._scan_weights(L, i, right, p + "mix.right.", n_att, lin, vec)
+                if m.branch_norm:
+                    L["left_out"], L["right_out"] = vec(p + "mix.left.out"), vec(p + "mix.right.out")
+                    if L["left_out"].numel() != W or L["right_out"].numel() != W:
+                        raise ValueError(f"layer {i}: branch norm weights do not fit the width")
+        else:
+            raise ValueError(f"layer {i}: mixer kind {ls.kind} is not wired into the parallel layout")
+        self.max_proj = max(self.max_proj, L["w_in"].shape[0])
+        if isinstance(f, MoeFfSpec):
+            if f.router == "table" or f.identity or f.shared_ff:
+                raise ValueError(f"layer {i}: table-routed, identity and shared experts are not wired into the parallel layout")
+            self._load_moe(L, i, f, lin, vec, get, p)
+        elif f is not None:
+            if f.act not in seqops.ACT_KINDS or seqops.ACT_KINDS[f.act] not in seqops.ACT_GATED:
+                raise ValueError(f"layer {i}: dense feed-forward activation {f.act} is not a gated kind")
+            gu = lin(p + "mlp.gate", p + "mlp.up")          # stored with alternating rows (gate j, up j): the pair meets in one warp
+            L["w_down"] = lin(p + "mlp.down")
+            if tuple(gu.shape) != (2 * f.ff, W) or tuple(L["w_down"].shape) != (W, f.ff):
+                raise ValueError(f"layer {i}: feed-forward tensor shapes do not fit the configuration")
+            L["w_gu"] = gu.view(2, f.ff, W).transpose(0, 1).reshape(2 * f.ff, W).contiguous()
+            self.weight_bytes += (L["w_gu"].numel() + L["w_down"].numel()) * 2
+            self.max_ff_inner, self.max_ff_proj = max(self.max_ff_inner, f.ff), max(self.max_ff_proj, 2 * f.ff)
+        return L
+
+    def _scan_weights(self, L, i: int, r: ScanSpec, rp: str, col: int, lin, vec) -> None:
+        """tensors of a selective scan whose [x | z] rows begin at column `col` of the layer's stacked projection (z passes silu there)"""
+        W, Cn, N, R = self.cfg.width, r.inner, r.state, r.dt_rank
+        if not 1 <= r.conv <= 8:
+            raise ValueError(f"layer {i}: 1 to 8 convolution taps")
+        L["xz_col"], L["silu"] = col, (col + Cn, col + 2 * Cn)
+        L["conv_w"], L["conv_b"] = vec(rp + "conv"), vec(rp + "conv.b")
+        L["w_x"], L["w_dt"], L["w_ro"] = lin(rp + "x"), lin(rp + "dt"), lin(rp + "o")
+        L["dt_b"], L["D"] = vec(rp + "dt.b"), vec(rp + "D")
+        A = -torch.exp(vec(rp + "A_log").double())
+        if tuple(L["conv_w"].shape) != (Cn, r.conv) or L["conv_b"].numel() != Cn or tuple(L["w_x"].shape) != (R + 2 * N, Cn) or tuple(L["w_dt"].shape) != (Cn, R) \
+                or tuple(L["w_ro"].shape) != (W, Cn) or L["dt_b"].numel() != Cn or L["D"].numel() != Cn or tuple(A.shape) != (Cn, N):
+            raise ValueError(f"layer {i}: selective-scan tensor shapes do not fit the configuration")
+        L["a2"] = (A * 1.4426950408889634).float().contiguous()      # the kernels raise 2, not e
+        L["scan"] = seqops.scan_desc(L["a2"], L["D"], L["dt_b"], L["w_dt"])
+        self.max_rinner, self.max_dbc, self.max_rank = max(self.max_rinner, Cn), max(self.max_dbc, R + 2 * N), max(self.max_rank, R)
+        self.weight_bytes += (L["w_x"].numel() + L["w_dt"].numel() + L["w_ro"].numel()) * 2
+
     def _load_moe(self, L, i: int, f: "MoeFfSpec", lin, vec, get, p: Optional[str] = None) -> None:
         """tensors of a mixture-of-experts feed-forward: router (rows of a shared expert's token gate stacked behind it) or table, stacked expert
         weights (gated kinds with alternating gate / up rows), the shared expert"""
@@ -909,6 +1060,11 @@ class LayeredModel:
             L["correction"] = vec(p + "mlp.correction") if f.correction else None
             if L["correction"] is not None and L["correction"].numel() != f.experts + f.identity:
                 raise ValueError(f"layer {i}: one correction per router output expected")
+            E = f.experts + f.identity
+            if f.groups > 1 and (E % f.groups or not 1 <= f.keep <= f.groups or f.keep * (E // f.groups) < f.top):
+                raise ValueError(f"layer {i}: router groups / top do not fit the expert count")
+            kind = {"sigmoid": seqops.ROUTE_SIGMOID, "softmax": seqops.ROUTE_SOFTMAX, "top_softmax": seqops.ROUTE_TOP_SOFTMAX}[f.router]
+            L["route"] = seqops.route_desc(E, f.groups, f.keep, f.top, kind, group_best=f.group_best, renorm=f.renorm, scale=f.route_scale, correction=L["correction"])
         else:
             raise ValueError(f"layer {i}: unknown router kind {f.router}")
         if gated:
@@ -985,6 +1141,13 @@ class LayeredModel:
                     L["rec_state"] = torch.zeros((max_seqs, right.width), **f32)
                     L["conv_state"] = torch.zeros((max_seqs, max(right.conv - 1, 1), right.width), **f32)
                 continue
+            if cfg.layout == "parallel" and ls.kind == "two_branch":
+                att, right = m.left, m.right
+                L["kpool"] = torch.zeros((max(1, num_blocks), block_size, att.kv_heads, att.dim), **f32)
+                L["vpool"] = torch.zeros((max(1, num_blocks), block_size, att.kv_heads, att.vdim), **f32)
+                L["scan_state"] = torch.zeros((max_seqs, right.inner, right.state), **f32)
+                L["conv_state"] = torch.zeros((max_seqs, max(right.conv - 1, 1), right.inner), **f32)
+                continue
             if ls.kind == "retention":
                 L["ret_state"] = torch.zeros((max_seqs, m.heads, m.dim, m.vdim), **f32)
             elif ls.kind == "latent_attention":       # one row [latent | rotated key part] per position; keys and values of all heads come out of it
@@ -1014,6 +1177,8 @@ class LayeredModel:
         seen = set()
         for L in self.layers:
             m = L["spec"].mixer
+            if self.cfg.layout == "parallel" and L["spec"].kind == "two_branch":
+                m = m.left
             if self.cfg.layout == "out_norm":
                 att = m if L["spec"].kind == "attention" else m.left
                 maps = 2 if att.diff is not None else 1
@@ -1052,8 +1217,12 @@ class LayeredModel:
                     need = max([need] + [seqops.attn_scratch_floats(T, 1, m.heads, m.kv_heads, m.vdim, keys) for T in range(1, cap + 1)])
         return need
 
+    def scan_scratch_floats(self, cap: int) -> int:
+        """floats of the work area of the selective scans, which run beside the attention"""
+        return max([0] + [seqops.scan_scratch_floats(cap, self.max_seqs, L["spec"].mixer.right.inner, L["spec"].mixer.right.state) for L in self.layers if "scan" in L])
+
     def cache_bytes(self) -> int:
-        keys = ("canon1_state", "canon2_state", "kpool", "vpool", "kpooled", "vpooled", "conv_state", "ssm_state", "shift_state", "ret_state", "rec_state", "delta_state")
+        keys = ("canon1_state", "canon2_state", "kpool", "vpool", "kpooled", "vpooled", "conv_state", "ssm_state", "shift_state", "ret_state", "rec_state", "delta_state", "scan_state")
         return sum(L[k].numel() * 4 for L in self.layers for k in keys if k in L)
 
     def _ctx_buffers(self, rows: int):
@@ -1145,6 +1314,8 @@ class LayeredModel:
             self._run_out(ws, T, B, R, debug_layers)
         elif self.cfg.layout == "sandwich":
             self._run_sandwich(ws, T, B, R, debug_layers)
+        elif self.cfg.layout == "parallel":
+            self._run_parallel(ws, T, B, R, debug_layers)
         else:
             self._run_streams(ws, T, B, R, sample, debug_layers)
         if R:
@@ -1456,6 +1627,108 @@ class LayeredModel:
         if R and (not n or debug_layers is not None):
             ops.sandwich_norm(x, cfg.eps, a_out=ws.fin[:R], fin_w=self.final_norm, rows=want)
 
+    def _run_parallel(self, ws: _Workspace, T: int, B: int, R: int, debug_layers: Optional[list]) -> None:
+        """parallel layers over one residual x (f32): mixer and feed-forward read the same normed input.  Between two layers ONE kernel: the mixer's branches with
+        their norms (or the deferred norm of a linear attention), the weighted sum of the experts' rows, the residual sum, the row added in front of a
+        pass, the next layer's norm and its input in the activation type; after the last one the final norm of the wanted rows."""
+        cfg, ops = self.cfg, seqops
+        st = self._desc(ws, T, B)
+        x, a, y, y2, y3 = ws.h[:T], ws.a[:T], ws.y[:T], ws.y2[:T], ws.y3[:T]
+        want = ws.view("want")[:R]
+        n = len(self.layers)
+        # The feed-forward does not wait for the mixer, nor a mixer's recurrent branch for its attention: they run on streams of their own (inside a
+        # captured decode step: parallel branches of the graph).  Not while operators are timed alone.
+        par = self.overlap_branches and self.dev.type == "cuda" and seqops.timeline is None
+        if par and self._side is None:
+            self._side, self._side2 = torch.cuda.Stream(self.dev), torch.cuda.Stream(self.dev)
+        main = torch.cuda.current_stream(self.dev) if par else None
+
+        def beside(stream, fn):
+            """fn on `stream` after what the main stream has queued so far; returns the event to wait for (None: it ran in line)"""
+            if not par:
+                fn()
+                return None
+            fork, done = torch.cuda.Event(), torch.cuda.Event()
+            fork.record(main)
+            stream.wait_event(fork)
+            with torch.cuda.stream(stream):
+                fn()
+                done.record(stream)
+            return done
+
+        def entering(i):
+            e = self.layers[i]["spec"].enter
+            return self.loop_step[e[1]] if e is not None and e[1] is not None else None
+
+        def ending(i):
+            """what the kernel that ends layer i leaves behind: the next layer's input, or the final norm of the wanted rows; with debug_layers x alone"""
+            if debug_layers is not None:
+                return dict(x_out=x)
+            if i + 1 < n:
+                return dict(x_out=x, a_out=a, fin_w=self.layers[i + 1]["norm1"], add_vec=entering(i + 1))
+            return dict(a_out=ws.fin[:R], fin_w=self.final_norm, rows=want)
+
+        ops.embed_pos(self.embed, ws.view("ids"), st, cfg.embed_scale, None, x, cfg.eps, add_vec=entering(0) if n else None, fin_w=self.layers[0]["norm1"] if n else None,
+                      a=a if n else None)
+        for i, L in enumerate(self.layers):
+            ls: LayerSpec = L["spec"]
+            m, f = ls.mixer, ls.ff
+            skip = debug_layers is None and i + 1 == n and not R       # nothing wanted: of the last layer only the cache and the state are needed
+            ff_done, close = None, {}
+            if f is not None and not skip:
+                if isinstance(f, MoeFfSpec):
+                    rows = {}
+                    ff_done = beside(self._side2, lambda: rows.update(self._moe_rows(L, f, ws, T, a)))
+                    close.update(rows)
+                else:
+                    ff_done = beside(self._side2, lambda: self._dense_ff(L, f, ws, T, a, y3, inner=ws.ff_inner, proj=ws.ff_proj))
+                    close["y3"] = y3
+            proj = ws.proj[:T, :L["w_in"].shape[0]]
+            ops.linear(a, L["w_in"], proj, silu=L["silu"])
+            if ls.kind == "retention":
+                H, V = m.heads, m.vdim
+                o = ws.inner_a.view(-1)[:T * H * V].view(T, H * V)
+                if m.norm == "joint":
+                    P = ops.retention_partials(T, B, H, V)
+                    close.update(sumsq=ws.sumsq.view(-1)[:T * P].view(T, P), sumsq_count=H * V)
+                ops.retention(proj, st, L["desc"], L["ret_state"], o, ws.scratch, sumsq=close.get("sumsq"))
+                ops.linear(o, L["w_o"], y)
+            elif ls.kind == "attention":
+                self._attention_out(L, m, ws, st, T, proj, y)
+            else:
+                right_done = beside(self._side, lambda: self._scan_branch(L, m.right, ws, st, T, proj, y2))
+                self._attention_out(L, m.left, ws, st, T, proj, y)
+                if right_done is not None:
+                    main.wait_event(right_done)
+                close.update(w_b1=L.get("left_out"), s1=m.left_scale, y2=y2, w_b2=L.get("right_out"), s2=m.right_scale)
+            if ff_done is not None:
+                main.wait_event(ff_done)
+            if skip:
+                break
+            ops.parallel_close(x, y, cfg.residual_mult, cfg.eps, **close, **ending(i))
+            if debug_layers is not None:
+                debug_layers.append(x.cpu())
+                if i + 1 < n:
+                    ops.sandwich_norm(x, cfg.eps, x_out=x, a_out=a, fin_w=self.layers[i + 1]["norm1"], add_vec=entering(i + 1))
+        if R and (not n or debug_layers is not None):
+            ops.sandwich_norm(x, cfg.eps, a_out=ws.fin[:R], fin_w=self.final_norm, rows=want)
+
+    def _scan_branch(self, L, r: ScanSpec, ws: _Workspace, st, T: int, proj: torch.Tensor, y: torch.Tensor) -> None:
+        Cn, N, R, c0 = r.inner, r.state, r.dt_rank, L["xz_col"]
+        u = ws.conv_a.view(-1)[:T * Cn].view(T, Cn)
+        seqops.causal_conv(proj[:, c0:c0 + Cn], L["conv_w"], L["conv_b"], L["conv_state"], st, seqops.CONV_SILU, u)
+        dbc = ws.dbc.view(-1)[:T * (R + 2 * N)].view(T, R + 2 * N)
+        seqops.linear(u, L["w_x"], dbc)
+        dtz = None
+        if st.T != st.B:        # portions: the step-size projection as one product; single tokens: inside the scan's kernel
+            low = ws.low.view(-1)[:T * R].view(T, R)
+            dtz = ws.dtz.view(-1)[:T * Cn].view(T, Cn)
+            seqops.act(dbc[:, :R], seqops.ACT_IDENT, low)
+            seqops.linear(low, L["w_dt"], dtz)
+        out = ws.inner_b.view(-1)[:T * Cn].view(T, Cn)
+        seqops.selective_scan(u, dbc, dtz, proj[:, c0 + Cn:c0 + 2 * Cn], st, L["scan"], L["scan_state"], out, ws.scratch_b)
+        seqops.linear(out, L["w_ro"], y)
+
     def _delta(self, L, m: DeltaSpec, ws: _Workspace, st, T: int, proj: torch.Tensor, y: torch.Tensor) -> None:
         H, D, V, d = m.heads, m.dim, m.vdim, L["desc"]
         o = ws.inner_a.view(-1)[:T * H * V].view(T, H * V)
@@ -1620,12 +1893,10 @@ class LayeredModel:
 
     MOE_ROW_PAIRS = 64      # up to this many (token, choice) pairs the experts' weights are streamed per pair; more: tiles over sorted pairs
 
-    def _moe_ff(self, L, f: "MoeFfSpec", ws: _Workspace, T: int, a: torch.Tensor, y: torch.Tensor, shared_done=None, route=None, x_id=None) -> None:
-        """shared_done: event after which the shared expert's output is in ws.moe_sh (it ran elsewhere); None: it runs here.
-        route: the layer's own choice buffers, filled (and sorted) earlier in the step (table-routed layers); None: the choice is made here"""
+    def _moe_rows(self, L, f: "MoeFfSpec", ws: _Workspace, T: int, a: torch.Tensor, route=None) -> dict:
+        """choice of the experts and their rows: the kernel that closes the layer sums them.  route: as in _moe_ff"""
         ops = seqops
         E, top = f.experts + f.identity, f.top      # E: router outputs (identity experts behind the real ones: they take part in the choice and the sort)
-        gated_shared = bool(f.shared_ff and f.shared_gate)
         pairs = T * top
         rows_form = pairs <= self.MOE_ROW_PAIRS
         z = None
@@ -1634,21 +1905,13 @@ class LayeredModel:
             pass
         elif f.router == "table":         # no router: the token id names the experts
             ops.moe_table_route(L["table"], ws.view("ids"), T, E, top, ids, wts, None if rows_form else ws.moe_cnt)
-        elif f.router in ("softmax", "top_softmax"):
-            kind = ops.ROUTE_SOFTMAX if f.router == "softmax" else ops.ROUTE_TOP_SOFTMAX
-            z = ws.moe_z[:T, :L["w_router"].shape[0]]
-            if T <= 8 and rows_form:        # few tokens: projection and choice in one kernel
-                ops.moe_router_ex(a, L["w_router"], E, 1, 1, top, kind, L["correction"], z, ids, wts)
-            else:
-                ops.linear(a, L["w_router"], z)
-                ops.moe_route_ex(z, E, 1, 1, top, kind, L["correction"], ids, wts, None if rows_form else ws.moe_cnt)
         else:
             z = ws.moe_z[:T, :L["w_router"].shape[0]]
             if T <= 8 and rows_form:        # few tokens: projection and choice in one kernel
-                ops.moe_router(a, L["w_router"], E, f.groups, f.keep, top, z, ids, wts)
+                ops.moe_router_rule(a, L["w_router"], L["route"], z, ids, wts)
             else:
                 ops.linear(a, L["w_router"], z)
-                ops.moe_route(z, E, f.groups, f.keep, top, ids, wts, None if rows_form else ws.moe_cnt)
+                ops.moe_route_rule(z, L["route"], ids, wts, None if rows_form else ws.moe_cnt)
         kind = ops.ACT_KINDS[f.act]
         mid = ws.moe_act.view(-1)[:pairs * f.ff].view(pairs, f.ff)
         act_args = (f.limit, f.alpha, f.up_shift) if kind in ops.ACT_GATED else ()     # gated experts: activation of the (gate, up) pairs in the projection's epilogue
@@ -1667,13 +1930,22 @@ class LayeredModel:
         else:
             ops.moe_linear(a, top, L["w_eup"], ids, order, offs, pairs, kind, mid, *act_args)
         ops.moe_linear(mid, 0, L["w_edown"], ids, order, offs, pairs, ops.ACT_NONE, ys)
+        return dict(ys=ys, wts=wts, slot_of=slot, top=top)
+
+    def _moe_ff(self, L, f: "MoeFfSpec", ws: _Workspace, T: int, a: torch.Tensor, y: torch.Tensor, shared_done=None, route=None, x_id=None) -> None:
+        """shared_done: event after which the shared expert's output is in ws.moe_sh (it ran elsewhere); None: it runs here.
+        route: the layer's own choice buffers, filled (and sorted) earlier in the step (table-routed layers); None: the choice is made here"""
+        ops = seqops
+        r = self._moe_rows(L, f, ws, T, a, route)
+        ys, wts, slot, top = r["ys"], r["wts"], r["slot_of"], r["top"]
+        ids = route["ids"] if route is not None else ws.moe_ids
+        gate_z = ws.moe_z[:T, f.experts + f.identity] if f.shared_ff and f.shared_gate and f.router != "table" else None
         sh = None
         if shared_done is not None:
             torch.cuda.current_stream(self.dev).wait_event(shared_done)
             sh = ws.moe_sh[:T]
         elif f.shared_ff:
             sh = self._shared_expert(L, f, ws, T, a)
-        gate_z = z[:, E] if gated_shared and z is not None else None
         if f.identity:
             ops.moe_combine_ex(ys, wts, slot, ids, f.experts, x_id, T, top, sh, gate_z, y)
         else:

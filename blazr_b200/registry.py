@@ -12,7 +12,7 @@ from __future__ import annotations
 import os
 from typing import Callable, Dict
 
-from . import fenorax, gemosun, pafelorn, teselix, vodelix
+from . import fenorax, gemosun, pafelorn, teselix, vodelix, zetunex
 from .layered import LayeredConfig, LayeredModel
 
 LAYERED: Dict[str, Callable[[dict], LayeredConfig]] = {}
@@ -28,6 +28,7 @@ register_layered(gemosun.ARCHITECTURE, gemosun.parse_config)
 register_layered(pafelorn.ARCHITECTURE, pafelorn.parse_config)
 register_layered(teselix.ARCHITECTURE, teselix.parse_config)
 register_layered(vodelix.ARCHITECTURE, vodelix.parse_config)
+register_layered(zetunex.ARCHITECTURE, zetunex.parse_config)
 
 
 class UnknownArchitecture(ValueError):

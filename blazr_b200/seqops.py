@@ -3,7 +3,8 @@ operators of layer-list models (stream mixing + grouped RMS norm, carried-state 
 over a paged KV pool, the state-space recurrence, gated activations, the depth-averaged residual, mixtures of experts, retention,
 latent attention, per-head projections, token shift + gated post-norm, the branch sum + output norm of two-branch mixers, the bigram
 embedding, PolyNorm, soft caps, differential attention, minGRU and real-gated linear recurrences, soft-max routing with identity experts,
-the delta rule with per-channel decays, layers normed on both sides with sinusoidal positions and a token-dependent addition, arg-max).
+the delta rule with per-channel decays, layers normed on both sides with sinusoidal positions and a token-dependent addition, the selective scan
+with a decay per channel and state, the residual of parallel layers, arg-max).
 
 Like blazr_b200/ops.py, PyTorch is plumbing only (device memory, streams); every compute call goes through ctypes.  The library
 is compiled on first use when it is missing (`ensure_built`): a fresh checkout needs nothing but nvcc.  There is no CPU
@@ -42,7 +43,8 @@ EXPORTS = ["b200seq_last_error", "b200seq_version", "b200seq_launch_count", "b20
            "b200seq_latent_prep", "b200seq_rotary", "b200seq_retention", "b200seq_retention_scratch_floats", "b200seq_token_shift", "b200seq_post_norm",
            "b200seq_moe_route_ex", "b200seq_moe_router_ex", "b200seq_moe_combine_ex", "b200seq_causal_conv_ex", "b200seq_embed_bigram", "b200seq_branch_norm", "b200seq_polynorm", "b200seq_softcap",
            "b200seq_diff_combine", "b200seq_min_gru", "b200seq_rg_lru", "b200seq_delta", "b200seq_delta_scratch_floats", "b200seq_embed_pos", "b200seq_sandwich_norm",
-           "b200seq_token_gate", "b200seq_side_close"]
+           "b200seq_token_gate", "b200seq_side_close", "b200seq_linear_silu", "b200seq_moe_route_rule", "b200seq_moe_router_rule", "b200seq_retention_partials",
+           "b200seq_selective_scan", "b200seq_scan_scratch_floats", "b200seq_parallel_close"]
 
 
 class SeqError(RuntimeError):
@@ -70,16 +72,17 @@ class RetentionDesc(C.Structure):
     """b200seq_retention_desc: sizes, columns of the projection row, decays and rotation constants of one retention layer"""
     _fields_ = [("H", C.c_int32), ("D", C.c_int32), ("V", C.c_int32), ("q_col", C.c_int32), ("k_col", C.c_int32), ("v_col", C.c_int32), ("g_col", C.c_int32),
                 ("decay", C.c_void_p), ("eps", C.c_float), ("rot_dims", C.c_int32), ("rot_half", C.c_int32), ("rot_freq", C.c_void_p), ("rot_scale", C.c_float),
-                ("k_scale", C.c_float)]
+                ("k_scale", C.c_float), ("norm_w", C.c_void_p), ("gate_sigmoid", C.c_int32), ("sumsq", C.c_void_p)]
 
 
 def retention_desc(H: int, D: int, V: int, decay: torch.Tensor, eps: float, k_scale: float, *, rot_freq: Optional[torch.Tensor] = None, rot_half: bool = True,
-                   rot_scale: float = 1.0) -> "RetentionDesc":
-    """descriptor for a projection row laid out q | k | v | gate; decay: device f32 [2, H] (decays, their base-2 logarithms); the caller
-    keeps decay and rot_freq alive"""
+                   rot_scale: float = 1.0, norm_w: Optional[torch.Tensor] = None, gate_sigmoid: bool = False) -> "RetentionDesc":
+    """descriptor for a projection row laid out q | k | v | gate; decay: device f32 [2, H] (decays, their base-2 logarithms); norm_w: f32 [H * V], one
+    norm over all heads, deferred (see include/b200seq.h); the caller keeps the tensors alive"""
     assert decay.dtype == torch.float32 and tuple(decay.shape) == (2, H) and decay.is_contiguous()
     d = RetentionDesc(H, D, V, 0, H * D, 2 * H * D, 2 * H * D + H * V, decay.data_ptr(), eps, 2 * rot_freq.numel() if rot_freq is not None else 0, int(rot_half),
-                      rot_freq.data_ptr() if rot_freq is not None else None, rot_scale, k_scale)
+                      rot_freq.data_ptr() if rot_freq is not None else None, rot_scale, k_scale, norm_w.data_ptr() if norm_w is not None else None, int(gate_sigmoid))
+    assert norm_w is None or (norm_w.dtype == torch.float32 and norm_w.numel() == H * V and norm_w.is_contiguous())
     d.width = 2 * H * D + 2 * H * V
     return d
 
@@ -287,12 +290,12 @@ def gated_act(gu: torch.Tensor, limit: float, alpha: float, up_shift: float, out
 
 
 @_timed
-def linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, path: int = PATH_AUTO):
-    """y[M, N] (f32) = x[M, K] . w[N, K]^T; w bf16 contiguous"""
+def linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, path: int = PATH_AUTO, silu: tuple = (0, 0)):
+    """y[M, N] (f32) = x[M, K] . w[N, K]^T; w bf16 contiguous; the columns silu[0] .. silu[1] - 1 of y pass silu"""
     M, K, ldx = _rows2d(x)
     _, N, ldy = _rows2d(y)
     assert w.dtype == torch.bfloat16 and w.is_contiguous() and tuple(w.shape) == (N, K) and y.dtype == torch.float32 and y.shape[0] == M
-    _check(lib().b200seq_linear(_p(x), _DT[x.dtype], C.c_int64(ldx), _p(w), M, N, K, _p(y), C.c_int64(ldy), path, _st(x)))
+    _check(lib().b200seq_linear_silu(_p(x), _DT[x.dtype], C.c_int64(ldx), _p(w), M, N, K, _p(y), C.c_int64(ldy), silu[0], silu[1], path, _st(x)))
 
 
 @_timed
@@ -491,9 +494,21 @@ def retention_scratch_floats(T: int, B: int, H: int, D: int, V: int) -> int:
     return int(f(T, B, H, D, V))
 
 
+def retention_partials(T: int, B: int, H: int, V: int) -> int:
+    """sums of squares a retention step with one norm over all heads leaves per token"""
+    return int(lib().b200seq_retention_partials(T, B, H, V))
+
+
 @_timed
-def retention(proj: torch.Tensor, step: "StepDesc", d: "RetentionDesc", state: torch.Tensor, out: torch.Tensor, scratch: Optional[torch.Tensor] = None):
+def retention(proj: torch.Tensor, step: "StepDesc", d: "RetentionDesc", state: torch.Tensor, out: torch.Tensor, scratch: Optional[torch.Tensor] = None,
+              sumsq: Optional[torch.Tensor] = None):
+    """sumsq: f32 [T, retention_partials] of a descriptor with one norm over all heads"""
     _, _, ld = _rows2d(proj)
+    if sumsq is not None:       # the descriptor of a call is a copy: the layer's own stays as it was
+        assert sumsq.dtype == torch.float32 and sumsq.is_contiguous() and sumsq.numel() >= step.T * retention_partials(step.T, step.B, d.H, d.V)
+        d2 = RetentionDesc.from_buffer_copy(d)
+        d2.sumsq = sumsq.data_ptr()
+        d = d2
     assert out.is_contiguous() and state.is_contiguous() and (scratch is None or (scratch.dtype == torch.float32 and scratch.is_contiguous()))
     _check(lib().b200seq_retention(_p(proj), C.c_int64(ld), C.byref(step), C.byref(d), _p(state), _p(out), _DT[out.dtype], _p(scratch),
                                    C.c_size_t(scratch.numel() if scratch is not None else 0), _st(proj)))
@@ -722,3 +737,91 @@ def side_close(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, ga
     assert gate.dtype == proj.dtype == table.dtype == torch.bfloat16 and table.is_contiguous()
     _check(lib().b200seq_side_close(_p(x), _p(y), _p(w), C.c_float(eps), _p(gate), _p(proj), _p(table), C.c_int64(table.shape[1]), col, dim, _p(ids), _p(side_w),
                                     _p(add_row), _p(add_vec), W, _p(rows), R, _p(x_out), _p(a_out), _DT[a_out.dtype] if a_out is not None else F32, _p(fin_w), _st(x)))
+
+
+# ---- routing with every constant given; selective scan; residual of parallel layers ------------------------------------------------------------
+class RouteDesc(C.Structure):
+    """b200seq_route_desc: sizes and constants of a router's choice"""
+    _fields_ = [("E", C.c_int32), ("groups", C.c_int32), ("keep", C.c_int32), ("top", C.c_int32), ("kind", C.c_int32), ("group_best", C.c_int32), ("renorm", C.c_int32),
+                ("scale", C.c_float), ("correction", C.c_void_p)]
+
+
+def route_desc(E: int, groups: int, keep: int, top: int, kind: int, *, group_best: int = 2, renorm: bool = True, scale: float = 1.0,
+               correction: Optional[torch.Tensor] = None) -> "RouteDesc":
+    """group_best: a group's score is the sum of its two largest scores (2) or its largest (1); renorm: weights divided by their sum; the caller keeps correction alive"""
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
+    return RouteDesc(E, groups, keep, top, kind, group_best, int(renorm), scale, correction.data_ptr() if correction is not None else None)
+
+
+@_timed
+def moe_route_rule(z: torch.Tensor, d: "RouteDesc", ids: torch.Tensor, wts: torch.Tensor, counts: Optional[torch.Tensor]):
+    T, _, ldz = _rows2d(z)
+    assert ids.dtype == torch.int32 and wts.dtype == torch.float32 and ids.is_contiguous() and wts.is_contiguous() and ids.numel() >= T * d.top
+    _check(lib().b200seq_moe_route_rule(_p(z), C.c_int64(ldz), T, C.byref(d), _p(ids), _p(wts), _p(counts), _st(z)))
+
+
+@_timed
+def moe_router_rule(x: torch.Tensor, w: torch.Tensor, d: "RouteDesc", z: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor):
+    """router projection and choice of at most 8 tokens in one kernel"""
+    T, K, ldx = _rows2d(x)
+    _, NR, ldz = _rows2d(z)
+    assert w.dtype == torch.bfloat16 and w.is_contiguous() and tuple(w.shape) == (NR, K) and z.dtype == torch.float32 and z.shape[0] == T
+    _check(lib().b200seq_moe_router_rule(_p(x), _DT[x.dtype], C.c_int64(ldx), _p(w), T, NR, K, C.byref(d), _p(z), C.c_int64(ldz), _p(ids), _p(wts), _st(x)))
+
+
+class ScanDesc(C.Structure):
+    """b200seq_scan_desc: sizes and weights of one selective scan"""
+    _fields_ = [("C", C.c_int32), ("N", C.c_int32), ("R", C.c_int32), ("a2", C.c_void_p), ("D", C.c_void_p), ("dt_b", C.c_void_p), ("w_dt", C.c_void_p)]
+
+
+def scan_desc(a2: torch.Tensor, D: torch.Tensor, dt_b: torch.Tensor, w_dt: torch.Tensor) -> "ScanDesc":
+    """a2 f32 [C, N] = A * log2(e); D, dt_b f32 [C]; w_dt bf16 [C, R]; the caller keeps the tensors alive"""
+    Cn, N = a2.shape
+    assert a2.dtype == D.dtype == dt_b.dtype == torch.float32 and w_dt.dtype == torch.bfloat16 and D.numel() == dt_b.numel() == w_dt.shape[0] == Cn
+    assert a2.is_contiguous() and D.is_contiguous() and dt_b.is_contiguous() and w_dt.is_contiguous()
+    return ScanDesc(Cn, N, w_dt.shape[1], a2.data_ptr(), D.data_ptr(), dt_b.data_ptr(), w_dt.data_ptr())
+
+
+def scan_scratch_floats(T: int, B: int, Cn: int, N: int) -> int:
+    """floats of work area a selective-scan step of T tokens in B entries wants (0: none)"""
+    f = lib().b200seq_scan_scratch_floats
+    f.restype = C.c_size_t
+    return int(f(T, B, Cn, N))
+
+
+@_timed
+def selective_scan(u: torch.Tensor, dbc: torch.Tensor, dtz: Optional[torch.Tensor], gate: torch.Tensor, step: "StepDesc", d: "ScanDesc", state: torch.Tensor, out: torch.Tensor,
+                   scratch: Optional[torch.Tensor] = None):
+    """u [T, C]; dbc f32 [T, R + 2 N]; dtz f32 [T, C] (steps with portions; overwritten); gate f32 [T, C] view, already activated; state f32 [slots, C, N]"""
+    T, _, ldd = _rows2d(dbc)
+    _, _, ldg = _rows2d(gate)
+    assert u.is_contiguous() and u.shape[1] == d.C and out.is_contiguous() and out.shape[1] == d.C and state.is_contiguous() and tuple(state.shape[1:]) == (d.C, d.N)
+    assert dbc.dtype == gate.dtype == state.dtype == torch.float32 and (dtz is None or (dtz.dtype == torch.float32 and dtz.is_contiguous() and dtz.shape[1] == d.C))
+    assert scratch is None or (scratch.dtype == torch.float32 and scratch.is_contiguous())
+    _check(lib().b200seq_selective_scan(_p(u), _DT[u.dtype], _p(dbc), C.c_int64(ldd), _p(dtz), _p(gate), C.c_int64(ldg), C.byref(step), C.byref(d), _p(state), _p(out),
+                                        _DT[out.dtype], _p(scratch), C.c_size_t(scratch.numel() if scratch is not None else 0), _st(dbc)))
+
+
+class ParallelDesc(C.Structure):
+    """b200seq_parallel_desc"""
+    _fields_ = [("x", C.c_void_p), ("y1", C.c_void_p), ("w_b1", C.c_void_p), ("ss1", C.c_void_p), ("ss_n", C.c_int32), ("ss_count", C.c_int32), ("s1", C.c_float),
+                ("y2", C.c_void_p), ("w_b2", C.c_void_p), ("s2", C.c_float), ("y3", C.c_void_p), ("ys", C.c_void_p), ("wts", C.c_void_p), ("slot_of", C.c_void_p),
+                ("top", C.c_int32), ("mult", C.c_float), ("add_vec", C.c_void_p), ("eps", C.c_float), ("W", C.c_int32), ("rows", C.c_void_p), ("R", C.c_int32),
+                ("x_out", C.c_void_p), ("a_out", C.c_void_p), ("out_dtype", C.c_int32), ("fin_w", C.c_void_p)]
+
+
+@_timed
+def parallel_close(x: torch.Tensor, y1: torch.Tensor, mult: float, eps: float, *, w_b1: Optional[torch.Tensor] = None, sumsq: Optional[torch.Tensor] = None, sumsq_count: int = 0,
+                   s1: float = 1.0, y2: Optional[torch.Tensor] = None, w_b2: Optional[torch.Tensor] = None, s2: float = 1.0, y3: Optional[torch.Tensor] = None,
+                   ys: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None, slot_of: Optional[torch.Tensor] = None, top: int = 0,
+                   add_vec: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, x_out: Optional[torch.Tensor] = None, a_out: Optional[torch.Tensor] = None,
+                   fin_w: Optional[torch.Tensor] = None):
+    """n = x + mult * (s1 b1 + s2 b2 + ff) + add_vec; b1 = y1, rms-normed with w_b1 or divided by the root of its deferred norm (sumsq [T, P], over sumsq_count
+    elements); b2 = y2 (rms-normed with w_b2); ff = y3 or the weighted sum of a token's expert rows ys; x_out = n, a_out = n (normed with fin_w when given)"""
+    W = x.shape[-1]
+    R = x.shape[0] if rows is None else rows.numel()
+    assert all(t is None or (t.is_contiguous() and t.dtype == torch.float32) for t in (x, y1, y2, y3, ys, wts, sumsq, x_out, add_vec)) and (a_out is None or a_out.is_contiguous())
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    d = ParallelDesc(ptr(x), ptr(y1), ptr(w_b1), ptr(sumsq), sumsq.shape[1] if sumsq is not None else 0, sumsq_count, s1, ptr(y2), ptr(w_b2), s2, ptr(y3), ptr(ys), ptr(wts),
+                     ptr(slot_of), top, mult, ptr(add_vec), eps, W, ptr(rows), R, ptr(x_out), ptr(a_out), _DT[a_out.dtype] if a_out is not None else F32, ptr(fin_w))
+    _check(lib().b200seq_parallel_close(C.byref(d), _st(x)))

@@ -30,7 +30,7 @@ from __future__ import annotations
 
 import math
 
-from .layered import AttentionSpec, DeltaSpec, DenseFfSpec, LayeredConfig, LayerSpec, MoeFfSpec
+from .layered import AttentionSpec, DeltaSpec, DenseFfSpec, LayeredConfig, LayerSpec, MoeFfSpec, loop_runs
 
 ARCHITECTURE = "Vodelix"
 POSITION_BASE = 10000.0
@@ -90,14 +90,11 @@ def _feed_forward(mlp, where: str):
 def layer_runs(n: int, loop) -> list:
     """(layer, pass or None outside the loop, first layer of its pass) in the order they run"""
     if loop is None:
-        return [(i, None, False) for i in range(n)]
+        return loop_runs(n)
     start, stop, times = (int(_need(loop, k, "loop")) for k in ("start", "stop", "times"))
     if not (0 <= start < stop <= n) or times < 1:
         raise ConfigError("config: loop: 0 <= start < stop <= number of layers, times >= 1")
-    runs = [(i, None, False) for i in range(start)]
-    for t in range(times):
-        runs += [(i, t, i == start) for i in range(start, stop)]
-    return runs + [(i, None, False) for i in range(stop, n)]
+    return loop_runs(n, start, stop, times)
 
 
 def parse_config(cfg: dict) -> LayeredConfig:

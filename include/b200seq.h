@@ -9,7 +9,8 @@
  * q / k norms, soft-capped scores, kept first positions, differential attention, minGRU and real-gated
  * linear recurrences, PolyNorm, soft-max routing with identity experts, a hashed bigram embedding,
  * the delta rule with per-channel decays, layers normed on both sides with sinusoidal positions and a
- * token-dependent addition, arg-max sampling.
+ * token-dependent addition, the selective scan with a decay per channel and state, the residual of parallel
+ * layers, arg-max sampling.
  *
  * It sits beside libb200q (include/b200q.h), which holds the quantized linear layer; the conventions are
  * the same:
@@ -105,6 +106,9 @@ int b200seq_gated_act(const float* gu, int64_t ldg, int T, int F, float limit, f
 
 /* y[M, N] (f32, stride ldy) = x[M, K] (f32 or bf16, stride ldx) . w[N, K]^T (bf16, contiguous) */
 int b200seq_linear(const void* x, int x_dtype, int64_t ldx, const void* w_bf16, int M, int N, int K, float* y, int64_t ldy, int path, void* stream);
+/* the same, and the columns [silu_lo, silu_hi) of y pass silu (a stacked projection some of whose parts feed a recurrence through silu) */
+int b200seq_linear_silu(const void* x, int x_dtype, int64_t ldx, const void* w_bf16, int M, int N, int K, float* y, int64_t ldy, int silu_lo, int silu_hi, int path,
+                        void* stream);
 
 /* Fused gate|up projection + gated activation: w_il is the stacked weight [2F, K] with rows alternating (gate 0, up 0, gate 1, up 1, ...);
  * out[M, F] (act dtype, stride ldo) = gated_act(x . w_il^T) with the formula of b200seq_gated_act.  The [M, 2F] product is never written.
@@ -258,7 +262,10 @@ int b200seq_rotary(float* x, int64_t ld, int col, int nheads, int D, const b200s
  * in steps of portions), k is multiplied by k_scale; per head with state[slot][H][D][V] (f32, read as zero when ent_pos0 == 0):
  *   S_t = decay[h] * S_(t-1) + k_t v_t^T;   o_t = S_t^T q_t;   out[t][h] = o_t / sqrt(mean(o_t^2) + eps) * silu(gate_t[h])   (act dtype [T, H*V])
  * decay: device f32 [2][H] = the decays, then their base-2 logarithms.  Steps in which every entry brings one token run one kernel and need
- * no work area; other steps cut the portions into chunks that run in parallel and need b200seq_retention_scratch_floats(...) floats. */
+ * no work area; other steps cut the portions into chunks that run in parallel and need b200seq_retention_scratch_floats(...) floats.
+ * With norm_w: ONE root mean square over all heads of a token, its division deferred.  out[t][h] = o_t * norm_w[h] * g(gate_t[h]) and sumsq[t][P]
+ * receives the squares of o_t, summed per head and tile of value columns (P = b200seq_retention_partials); whoever reads what the linear layer made
+ * of out multiplies the row by 1 / sqrt(sum_P sumsq[t] / (H V) + eps) (b200seq_parallel_close does). */
 typedef struct b200seq_retention_desc {
     int32_t H, D, V;
     int32_t q_col, k_col, v_col, g_col;
@@ -267,7 +274,12 @@ typedef struct b200seq_retention_desc {
     int32_t rot_dims, rot_half;
     const float* rot_freq;
     float rot_scale, k_scale;
+    /* ---- fields below default to zero / null ---- */
+    const float* norm_w;   /* device f32 [H * V] or null: one norm over all heads, deferred */
+    int32_t gate_sigmoid;  /* 1: g = sigmoid instead of silu */
+    float* sumsq;          /* with norm_w: device f32 [T][P] */
 } b200seq_retention_desc;
+int b200seq_retention_partials(int T, int B, int H, int V);
 size_t b200seq_retention_scratch_floats(int T, int B, int H, int D, int V);
 int b200seq_retention(float* proj, int64_t ld, const b200seq_step* st, const b200seq_retention_desc* d, float* state, void* out, int out_dtype, float* scratch,
                       size_t scratch_floats, void* stream);
@@ -330,6 +342,17 @@ int b200seq_moe_route_ex(const float* z, int64_t ldz, int T, int E, int groups, 
 /* b200seq_moe_router with the score kind and correction of b200seq_moe_route_ex */
 int b200seq_moe_router_ex(const void* x, int x_dtype, int64_t ldx, const void* w_bf16, int T, int NR, int K, int E, int groups, int keep, int top, int kind,
                           const float* correction, float* z, int64_t ldz, int32_t* ids, float* wts, void* stream);
+/* The choice with every constant given: group_best 2 = a group's score is the sum of its two largest s, 1 = its largest; renorm 1 = the weights are
+ * scale * s / (sum of the chosen s + 1e-20), 0 = scale * s (not with kind 2).  (_route_ex / _router_ex: 2, 1, scale 1.) */
+typedef struct b200seq_route_desc {
+    int32_t E, groups, keep, top, kind;
+    int32_t group_best, renorm;
+    float scale;
+    const float* correction;
+} b200seq_route_desc;
+int b200seq_moe_route_rule(const float* z, int64_t ldz, int T, const b200seq_route_desc* d, int32_t* ids, float* wts, int32_t* counts, void* stream);
+int b200seq_moe_router_rule(const void* x, int x_dtype, int64_t ldx, const void* w_bf16, int T, int NR, int K, const b200seq_route_desc* d, float* z, int64_t ldz,
+                            int32_t* ids, float* wts, void* stream);
 /* b200seq_moe_combine with identity experts: a pair whose expert id is >= E_real has no row in ys; its output is the token's own input
  * x_id[t] (f32 [T, W]) times the weight.  ids: [T * top]. */
 int b200seq_moe_combine_ex(const float* ys, const float* wts, const int32_t* slot_of, const int32_t* ids, int E_real, const float* x_id, int T, int top, int W,
@@ -420,6 +443,51 @@ int b200seq_token_gate(const float* z, int64_t ldz, int T, int dim, const void* 
 int b200seq_side_close(const float* x, const float* y, const float* w, float eps, const void* gate_bf16, const void* proj_bf16, const void* table_bf16, int64_t ldt, int col,
                        int dim, const int32_t* ids, const float* side_w, const float* add_row, const float* add_vec, int W, const int32_t* rows, int R,
                        float* x_out, void* a_out, int out_dtype, const float* fin_w, void* stream);
+
+/* ---- selective scan with a decay per channel and state --------------------------------------------------------------------------------------------
+ * Per channel c < C and state n < N, with state[slot][C][N] (f32, read as zero when ent_pos0 == 0):
+ *   dt = softplus(z + dt_b[c]);  S <- exp(dt A) S + dt u B[n];  y = sum_n S C[n] + D[c] u;  out[t][c] = y * gate[t][c]      (act dtype [T, C])
+ * a2: f32 [C][N] = A * log2(e), A < 0.  u: [T, C] in u_dtype, contiguous.  rows dbc f32 (stride ldd): [low (R) | B (N) | C (N)].  gate: f32 rows (stride ldg),
+ * already activated.  z: steps in which every entry brings one token compute it themselves, z[t][c] = w_dt[c] . low[t] (w_dt bf16 [C][R]); other steps read it
+ * from dtz (f32 [T, C], contiguous), which a step of more than one segment overwrites with dt.  Steps with portions need b200seq_scan_scratch_floats(...)
+ * floats (0: none): segments of every portion run in parallel from a zero state, are combined in order and run again from their start states. */
+typedef struct b200seq_scan_desc {
+    int32_t C, N, R;
+    const float *a2, *D, *dt_b;
+    const void* w_dt;
+} b200seq_scan_desc;
+size_t b200seq_scan_scratch_floats(int T, int B, int C, int N);
+int b200seq_selective_scan(const void* u, int u_dtype, const float* dbc, int64_t ldd, float* dtz, const float* gate, int64_t ldg, const b200seq_step* st,
+                           const b200seq_scan_desc* d, float* state, void* out, int out_dtype, float* scratch, size_t scratch_floats, void* stream);
+
+/* ---- residual path of parallel layers: mixer and feed-forward read the same normed input ------------------------------------------------------------
+ * One block per row r (token t = rows ? rows[r] : r):
+ *   b1 = w_b1 ? rms_norm(y1[t], eps) * w_b1 : (ss1 ? y1[t] / sqrt(sum(ss1[t][0 .. ss_n)) / ss_count + eps) : y1[t]);   b2 likewise from y2 with w_b2 (y2 optional)
+ *   f  = y3[t] (optional), or with ys: sum_(j < top) wts[t * top + j] * ys[slot_of ? slot_of[t * top + j] : t * top + j]      (the experts' rows)
+ *   n  = x[t] + mult * (s1 * b1 + s2 * b2 + f) + add_vec
+ *   x_out[t] <- n (optional, may be x);   a_out[r] <- fin_w ? rms_norm(n, eps) * fin_w : n, in out_dtype (optional)
+ * Everything in f32. */
+typedef struct b200seq_parallel_desc {
+    const float *x, *y1, *w_b1, *ss1;
+    int32_t ss_n, ss_count;
+    float s1;
+    const float *y2, *w_b2;
+    float s2;
+    const float *y3, *ys, *wts;
+    const int32_t* slot_of;
+    int32_t top;
+    float mult;
+    const float* add_vec;
+    float eps;
+    int32_t W;
+    const int32_t* rows;
+    int32_t R;
+    float* x_out;
+    void* a_out;
+    int32_t out_dtype;
+    const float* fin_w;
+} b200seq_parallel_desc;
+int b200seq_parallel_close(const b200seq_parallel_desc* d, void* stream);
 
 /* ids[r] = argmax_v logits[r][v] (first maximum) */
 int b200seq_argmax(const float* logits, int R, int V, int32_t* ids, void* stream);
