@@ -76,6 +76,43 @@ __global__ void embed_pos_kernel(const EmbedPos p, const b200seq_step st) {
     for (int j = threadIdx.x; j < W; j += blockDim.x) store_act(p.a, p.a_dtype, (int64_t)t * W + j, p.fin_w ? row[j] * rinv * p.fin_w[j] : row[j]);
 }
 
+// the same without positions, the row in registers (W % 4 == 0, W <= 4 * EPT * blockDim.x, 16-byte aligned rows)
+template <int EPT>
+__global__ void __launch_bounds__(512) embed_reg_kernel(const EmbedPos p) {
+    __shared__ float red[40];
+    const int t = blockIdx.x, W = p.W, nt = blockDim.x;
+    const __nv_bfloat16* src = p.table + (int64_t)p.ids[t] * W;
+    float4 v[EPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < EPT; ++k) {
+        const int i = 4 * (threadIdx.x + k * nt);
+        v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i >= W) continue;
+        const uint2 r = *reinterpret_cast<const uint2*>(src + i);
+        v[k] = make_float4(__uint_as_float(r.x << 16) * p.scale, __uint_as_float(r.x & 0xffff0000u) * p.scale, __uint_as_float(r.y << 16) * p.scale,
+                           __uint_as_float(r.y & 0xffff0000u) * p.scale);
+        if (p.x0) *reinterpret_cast<float4*>(p.x0 + (int64_t)t * W + i) = v[k];
+        if (p.add_vec) v[k] = add4(v[k], ld4(p.add_vec + i));
+        *reinterpret_cast<float4*>(p.x + (int64_t)t * W + i) = v[k];
+        ss = sq4(v[k], ss);
+    }
+    if (!p.a) return;
+    float rinv = 1.f;
+    if (p.fin_w) rinv = 1.0f / sqrtf(block_sum(ss, red) / (float)W + p.eps);
+#pragma unroll
+    for (int k = 0; k < EPT; ++k) {
+        const int i = 4 * (threadIdx.x + k * nt);
+        if (i >= W) continue;
+        float4 n = v[k];
+        if (p.fin_w) {
+            const float4 f = ld4(p.fin_w + i);
+            n = make_float4(n.x * rinv * f.x, n.y * rinv * f.y, n.z * rinv * f.z, n.w * rinv * f.w);
+        }
+        store_act4(p.a, p.a_dtype, (int64_t)t * W + i, n);
+    }
+}
+
 // ---- norm of a sublayer's result + residual + additions + next norm ----------------------------------------------------------------------------
 struct SandwichArgs {
     const float *x, *y, *w;
@@ -381,6 +418,16 @@ int b200seq_embed_pos(const void* table_bf16, const int32_t* ids, const b200seq_
     }
     const EmbedPos p{(const __nv_bfloat16*)table_bf16, ids, freq, scale, W, x0, add_vec, x, fin_w, eps, a, a_dtype,
                      W % 2 == 0 && ((reinterpret_cast<uintptr_t>(table_bf16) & 3) | (reinterpret_cast<uintptr_t>(x) & 7) | (reinterpret_cast<uintptr_t>(x0) & 7)) == 0};
+    auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    if (!freq && W % 4 == 0 && W <= 8192 && (reinterpret_cast<uintptr_t>(table_bf16) & 7) == 0 && al(x0) && al(add_vec) && al(x) && al(fin_w) && al(a)) {
+        const int q = W / 4, nt = q <= 64 ? 64 : (q <= 256 ? 128 : (q <= 1024 ? 256 : 512));
+        const int ept = (q + nt - 1) / nt;
+        if (ept <= 1) embed_reg_kernel<1><<<st->T, nt, 0, (cudaStream_t)stream>>>(p);
+        else if (ept <= 2) embed_reg_kernel<2><<<st->T, nt, 0, (cudaStream_t)stream>>>(p);
+        else embed_reg_kernel<4><<<st->T, nt, 0, (cudaStream_t)stream>>>(p);
+        SEQ_LAUNCH_CHECK("embed_pos");
+        return 0;
+    }
     embed_pos_kernel<<<st->T, W >= 1024 ? 512 : 128, smem, (cudaStream_t)stream>>>(p, *st);
     SEQ_LAUNCH_CHECK("embed_pos");
     return 0;

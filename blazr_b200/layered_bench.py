@@ -6,14 +6,16 @@ dense-attention decoder (blazr_b200/decode.py, Q8_0 weights) of the same width, 
     kernels  : every operator of one prefill step and one decode step timed alone (CUDA events around each launch), with its
                algorithmic bytes / FLOPs and the fraction of the roofline it reaches; the like kernels of the decoder beside them
 
-`python bench.py --layered fenorax|gemosun|teselix|pafelorn|vodelix [--layered-sizes w1024,w2048]` prints the result as one JSON line; bench.py's default
+`python bench.py --layered fenorax|gemosun|teselix|pafelorn|vodelix|zetunex [--layered-sizes w1024,w2048]` prints the result as one JSON line; bench.py's default
 workload and JSON line are untouched.  For Gemosun (parallel attention / feed-forward layers, three of four feed-forwards a mixture of
 experts) the closest existing model, Fenorax at the same sizes, runs beside it as well; for Teselix (retention and latent-attention mixers,
 table-routed experts) both run beside it: Gemosun is the closest in attention and experts, Fenorax in the recurrence.  For Pafelorn (windowed
 attention beside element-wise recurrences, differential attention, soft-max-routed gated experts) Gemosun (windowed attention with rotation,
 routed experts) and Fenorax (a recurrence with carried state and a short convolution) run beside it as well.  For Vodelix (a delta rule with a
 matrix state per head, unmasked causal attention, routed plain experts) Teselix (retention: a matrix state per head; experts) and Gemosun (plain
-experts behind a learned router) run beside it as well.
+experts behind a learned router) run beside it as well.  For Zetunex (parallel layers: linear attention with fixed decays, windowed attention beside a
+selective scan, routed gated experts) Teselix (retention), Fenorax (a state-space scan behind a short convolution) and Gemosun (parallel layers,
+windowed attention, experts behind a learned router) run beside it as well.
 """
 from __future__ import annotations
 
@@ -108,6 +110,56 @@ def vodelix_config(sz: dict, experts: int = 32, top: int = 4) -> dict:
     att = {"type": "attention", "mixer": {"heads": H, "kv_heads": sz["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5}}
     return {"architecture": "Vodelix", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "token_side": {"dim": W // 16}, "loop": {"start": 1, "stop": 2, "times": 2},
             "layers": [dict(delta, mlp={"kind": "dense", "ff": sz["ff"]}), dict(att, mlp=moe), dict(delta, mlp=dict(moe))]}
+
+
+def zetunex_config(sz: dict, experts: int = 32, top: int = 4, state: int = 16) -> dict:
+    """four runs of three parallel layers [attention | selective scan + dense, linear attention + experts (twice), attention | selective scan + experts] of the
+    size's width and head layout; windows of `chunk` positions; the scan is twice as wide as the model; an expert is a quarter of the dense size"""
+    H, D, W = sz["heads"], sz["dim"], sz["width"]
+    moe = {"kind": "moe", "expert": {"ff": sz["ff"] // 4}, "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    two = {"type": "parallel", "mixer": {"left": {"heads": H, "kv_heads": sz["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": sz["chunk"]}},
+                                         "right": {"inner": 2 * W, "state": state, "conv": 4, "dt_rank": W // 16}}}
+    lin = {"type": "lightning", "mixer": {"heads": H, "dim": D, "vdim": D, "decay": [1.0 - 2.0 ** (-5.0 - 7.0 * h / max(H - 1, 1)) for h in range(H)]}}
+    return {"architecture": "Zetunex", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "loop": {"start": 1, "stop": 2, "times": 2},
+            "layers": [dict(two, mlp={"kind": "dense", "ff": sz["ff"]}), dict(lin, mlp=moe), dict(two, mlp=dict(moe))]}
+
+
+def random_tensors_zetunex(cfg: dict, device, seed: int = 7):
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def rnd(*shape, scale=1.0):
+        return (torch.randn(shape, generator=g, device=device) * scale).to(torch.bfloat16)
+
+    ones = lambda *s: torch.ones(*s, dtype=torch.bfloat16, device=device)
+    t = {"embed": rnd(V, W), "final.norm": ones(W), "loop.step": rnd(cfg["loop"]["times"], W, scale=0.1)}
+    lin = lambda name, o, i: t.__setitem__(name, rnd(o, i, scale=i ** -0.5))
+    for i, lay in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", lay["mixer"], lay["mlp"]
+        t[p + "norm1"] = ones(W)
+        if lay["type"] == "lightning":
+            H, D, Vd = m["heads"], m["dim"], m["vdim"]
+            lin(p + "mix.q", H * D, W), lin(p + "mix.k", H * D, W), lin(p + "mix.v", H * Vd, W), lin(p + "mix.g", H * Vd, W), lin(p + "mix.o", W, H * Vd)
+            t[p + "mix.norm"] = ones(H * Vd)
+        else:
+            a, r = m["left"], m["right"]
+            for nm, o in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                lin(p + "mix.left." + nm, o, W)
+                t[p + "mix.left." + nm + ".b"] = rnd(o, scale=0.1)
+            lin(p + "mix.left.o", W, a["heads"] * a["vdim"])
+            C, N, R, q = r["inner"], r["state"], r["dt_rank"], p + "mix.right."
+            lin(q + "in", 2 * C, W), lin(q + "x", R + 2 * N, C), lin(q + "dt", C, R), lin(q + "o", W, C)
+            t[q + "conv"], t[q + "conv.b"], t[q + "dt.b"], t[q + "D"] = rnd(C, r["conv"], scale=0.5), rnd(C, scale=0.1), rnd(C) - 3.0, ones(C)
+            t[q + "A_log"] = torch.log(torch.arange(1, N + 1, device=device).float()).expand(C, N).to(torch.bfloat16).contiguous()
+            t[p + "mix.left.out"], t[p + "mix.right.out"] = ones(W), ones(W)
+        if f["kind"] == "dense":
+            lin(p + "mlp.gate", f["ff"], W), lin(p + "mlp.up", f["ff"], W), lin(p + "mlp.down", W, f["ff"])
+        else:
+            lin(p + "mlp.router", f["router"]["experts"], W)
+            for e in range(f["router"]["experts"]):
+                lin(p + f"mlp.e{e}.gate", f["expert"]["ff"], W), lin(p + f"mlp.e{e}.up", f["expert"]["ff"], W), lin(p + f"mlp.e{e}.down", W, f["expert"]["ff"])
+    return lambda name: t[name].cpu()
 
 
 def random_tensors_vodelix(cfg: dict, device, seed: int = 7, rank: int = 64):
@@ -322,7 +374,7 @@ def _events():
 
 def _linear_weights(model: LayeredModel) -> int:
     """weights of the linear layers a token goes through (of a mixture of experts: the router, the chosen experts, the shared one)"""
-    n = sum(L[k].numel() for L in model.layers for k in ("w_in", "w_o", "w_gu", "w_down", "w_router", "w_sup", "w_sdown", "rg1", "rg2", "w_uq", "w_ukT", "w_uv", "w_up", "w_ro", "w_gates", "w_2", "side_gate", "side_proj") if k in L)
+    n = sum(L[k].numel() for L in model.layers for k in ("w_in", "w_o", "w_gu", "w_down", "w_router", "w_sup", "w_sdown", "rg1", "rg2", "w_uq", "w_ukT", "w_uv", "w_up", "w_ro", "w_gates", "w_2", "side_gate", "side_proj", "w_x", "w_dt") if k in L)
     for L in model.layers:
         if "w_eup" in L:
             n += L["spec"].ff.top * (L["w_eup"][0].numel() + L["w_edown"][0].numel())
@@ -334,7 +386,7 @@ def _touched_bytes(model: LayeredModel, B: int) -> int:
     are touched) and the per-token table; layers that run several times count every time"""
     n = model.weight_bytes - (model.side_table.numel() * 2 if model.side_table is not None else 0)
     for L in model.layers:
-        if L["spec"].weights_of is not None and model.cfg.layout == "sandwich":
+        if L["spec"].weights_of is not None and model.cfg.layout in ("sandwich", "parallel"):
             n += 2 * sum(v.numel() for k, v in L.items() if isinstance(v, torch.Tensor) and v.dtype == torch.bfloat16)
         if "w_eup" in L:
             E_, per = L["w_eup"].shape[0], (L["w_eup"][0].numel() + L["w_edown"][0].numel()) * 2
@@ -397,6 +449,19 @@ def _cost(name: str, shapes, scal, scen: dict, kw: dict = None):
         W = sh[0][0][1]
         outs = sum(kw[n][1] for n in ("x_out", "a_out") if isinstance(kw.get(n), tuple))
         return rows * W * (8 + outs) + by(sh[3]) + by(sh[4]), 0.0, "hbm"
+    if name == "parallel_close":  # x, the branches, the feed-forward's rows in; x and / or the activation rows out
+        rows = kw["rows"][0][0] if isinstance(kw.get("rows"), tuple) else sh[0][0][0]
+        W = sh[0][0][1]
+        reads = 2 + sum(1 for n in ("y2", "y3") if isinstance(kw.get(n), tuple)) + (kw.get("top", 0) if isinstance(kw.get("ys"), tuple) else 0)
+        outs = sum(kw[n][1] for n in ("x_out", "a_out") if isinstance(kw.get(n), tuple))
+        return rows * W * (4 * reads + outs) + (by(kw["sumsq"]) if isinstance(kw.get("sumsq"), tuple) else 0), 0.0, "hbm"
+    if name == "selective_scan":  # u, the step sizes (portions: their product), gate and [low | B | C] rows in, the gated result out, the state of every entry read and written
+        d = scen["scan_desc"]
+        (T, Cn), ue = sh[0]
+        oe = next(s[1] for s in reversed(sh) if s[0] == (T, Cn))
+        rows = T * (Cn * (ue + 4 + oe + (4 if scen["prefill"] else 0)) + (d.R + 2 * d.N) * 4)
+        # decay (product, exponential), two products of the input, state update, output: the plain recurrence
+        return rows + Cn * d.N * 4 * (2 * scen["entries"] + 1) + (0 if scen["prefill"] else Cn * d.R * 2), 7.0 * T * Cn * d.N, "f32" if scen["prefill"] else "hbm"
     if name == "token_gate":      # logits and table rows in, gated rows out
         (T, dim) = sh[0][0]
         return T * dim * (4 + 2 + sh[-1][1]), 0.0, "hbm"
@@ -526,22 +591,26 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
     elif design.lower() == "vodelix":
         cfg = vodelix_config(sz)
         model = LayeredModel(registry.LAYERED["Vodelix"](cfg), random_tensors_vodelix(cfg, dev, rank={1024: 64, 2048: 96}.get(sz["width"], 128)), dev, dtype)
+    elif design.lower() == "zetunex":
+        cfg = zetunex_config(sz)
+        model = LayeredModel(registry.LAYERED["Zetunex"](cfg), random_tensors_zetunex(cfg, dev), dev, dtype)
     else:
         raise ValueError(f"no synthetic workload for design '{design}'")
-    gem, tes, paf, vod = (design.lower() == n for n in ("gemosun", "teselix", "pafelorn", "vodelix"))
+    gem, tes, paf, vod, zet = (design.lower() == n for n in ("gemosun", "teselix", "pafelorn", "vodelix", "zetunex"))
     pool = 16 if gem else 0
     desc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.AttnDesc)), None)
     rdesc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.RetentionDesc)), None)
     ddesc0 = next((L["desc"] for L in model.layers if isinstance(L.get("desc"), seqops.DeltaDesc)), None)
+    sdesc0 = next((L["scan"] for L in model.layers if "scan" in L), None)
     Bmax = max(batches)
     eng = Engine(model, max_tokens=max(S, Bmax * (ctx + steps + 64)) + 64, max_seqs=Bmax, max_step_tokens=max(S, 2048), prefill_chunk=S)
     rng = np.random.default_rng(3)
     prompt = rng.integers(0, sz["vocab"], S).tolist()
     out = {"size": size, "config": {k: sz[k] for k in sz}, "layers": [l["type"] + ("+" + l["mlp"].get("kind", "ff") if l["mlp"] else "") for l in cfg["layers"]],
            "streams": cfg.get("streams", 1), "linear_weights": _linear_weights(model), "weight_bytes": model.weight_bytes}
-    if gem or tes or paf or vod:
+    if gem or tes or paf or vod or zet:
         r = cfg["layers"][1]["mlp"]
-        out["experts"] = {"experts": r["router"]["experts"], "top": r["router"]["top"], "ff": r["expert"]["ff"], "shared_ff": r["shared"]["ff"], "groups": r["router"].get("groups")}
+        out["experts"] = {"experts": r["router"]["experts"], "top": r["router"]["top"], "ff": r["expert"]["ff"], "shared_ff": r["shared"]["ff"] if "shared" in r else 0, "groups": r["router"].get("groups")}
     lin_flops_tok = 2.0 * (_linear_weights(model) + 0)
 
     # prefill: whole prompt in one step, logits of the last token, device timed; then through run_entries (host arrays in, logits out)
@@ -576,8 +645,8 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
         scen = dict(prefill=True, entries=1, visible_keys=int(vis.sum()), kv_rows_touched=S + S // pool, attn_desc=desc0)
     elif vod:   # every earlier position
         scen = dict(prefill=True, entries=1, visible_keys=int((pos + 1).sum()), kv_rows_touched=S, attn_desc=desc0, delta_desc=ddesc0)
-    elif paf:   # a sliding window of `chunk` positions (the few kept first positions of one layer are not counted)
-        scen = dict(prefill=True, entries=1, visible_keys=int(np.minimum(pos + 1, chunk).sum()), kv_rows_touched=S, attn_desc=desc0)
+    elif paf or zet:   # a sliding window of `chunk` positions (the few kept first positions of one layer are not counted)
+        scen = dict(prefill=True, entries=1, visible_keys=int(np.minimum(pos + 1, chunk).sum()), kv_rows_touched=S, attn_desc=desc0, ret_desc=rdesc0, scan_desc=sdesc0)
     elif tes:   # every earlier position; a step of portions attends over per-head keys projected from the gathered latents
         descx = next((L["desc_x"] for L in model.layers if "desc_x" in L), desc0)
         scen = dict(prefill=True, entries=1, visible_keys=int((pos + 1).sum()), kv_rows_touched=S, attn_desc=descx, ret_desc=rdesc0)
@@ -621,8 +690,8 @@ def bench_layered(design: str, size: str, pk, S: int = 4096, ctx: int = 1024, ba
                "frac_hbm_weights_only": round(touched / (msd * 1e-3) / 1e9 / pk["hbm_gbs"], 3)}
         held = eng.cache.live[ids[0]].n_tokens
         lo = (held // chunk) * chunk
-        seen = (min(held + 1, chunk) + max(0, (held - chunk + 1) // pool)) if gem else (held + 1 if tes or vod else (min(held + 1, chunk) if paf else held - lo + 1))
-        scen = dict(prefill=False, entries=B, visible_keys=B * seen, kv_rows_touched=B * seen, attn_desc=desc0, ret_desc=rdesc0, delta_desc=ddesc0)
+        seen = (min(held + 1, chunk) + max(0, (held - chunk + 1) // pool)) if gem else (held + 1 if tes or vod else (min(held + 1, chunk) if paf or zet else held - lo + 1))
+        scen = dict(prefill=False, entries=B, visible_keys=B * seen, kv_rows_touched=B * seen, attn_desc=desc0, ret_desc=rdesc0, delta_desc=ddesc0, scan_desc=sdesc0)
         row["kernels"] = kernel_table(model, eng, dec_step, scen, pk)
         out["decode"].append(row)
         for r in ids:
@@ -778,7 +847,7 @@ def run(design: str, sizes: List[str], pk, pk_kind: str, S: int = 4096, ctx: int
     for size in sizes:
         row = {"size": size}
         row[design.lower()] = bench_layered(design, size, pk, S=S, ctx=ctx, steps=steps)
-        others = {"fenorax": [], "gemosun": ["fenorax"], "teselix": ["gemosun", "fenorax"], "pafelorn": ["gemosun", "fenorax"], "vodelix": ["teselix", "gemosun"]}.get(design.lower(), ["fenorax"])
+        others = {"fenorax": [], "gemosun": ["fenorax"], "teselix": ["gemosun", "fenorax"], "pafelorn": ["gemosun", "fenorax"], "vodelix": ["teselix", "gemosun"], "zetunex": ["teselix", "fenorax", "gemosun"]}.get(design.lower(), ["fenorax"])
         for other in others:                # the closest existing layer-list models at the same sizes
             try:
                 row[other] = bench_layered(other, size, pk, S=S, ctx=ctx, steps=steps)
