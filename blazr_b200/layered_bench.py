@@ -410,7 +410,8 @@ def _cost(name: str, shapes, scal, scen: dict, kw: dict = None):
         d = scen.get("attn_desc")
         T, ld = sh[0][0]
         if name == "attn_prep_ex" and d is not None:
-            return T * (ld + d.H * d.D + d.G * (d.D + d.V)) * 4, 0.0, "hbm"
+            cols = d.H * d.D + d.G * (d.D + d.V)       # the row may hold other parts of the layer's stacked projection
+            return T * (min(ld, cols) + cols) * 4, 0.0, "hbm"
         return T * ld * 4 * 2, 0.0, "hbm"
     if name in ("linear", "linear_gated", "linear_act"):
         (xs, xe), (ws, _), (ys, ye) = sh[0], sh[1], sh[2]
@@ -465,6 +466,9 @@ def _cost(name: str, shapes, scal, scen: dict, kw: dict = None):
     if name == "token_gate":      # logits and table rows in, gated rows out
         (T, dim) = sh[0][0]
         return T * dim * (4 + 2 + sh[-1][1]), 0.0, "hbm"
+    if name == "embed_streams":   # table rows in, every stream out
+        (T, S_, W) = sh[-1][0]
+        return T * W * (2 + 4 * S_), 0.0, "hbm"
     if name == "embed_pos":       # table rows in; x, the embedding output and the activation rows out
         (T, W) = sh[-1][0]
         return T * W * (2 + 4 + sum(kw[n][1] for n in ("x0", "a") if isinstance(kw.get(n), tuple))), 0.0, "hbm"
