@@ -220,6 +220,33 @@ __global__ void attn_prep_gen_kernel(float* __restrict__ proj, int64_t ld, b200s
     }
 }
 
+// The general form when all it has to do is add the bias: grid (T, slices of the q | k | v columns), VW columns per thread
+template <int VW>
+__global__ void attn_prep_bias_kernel(float* __restrict__ proj, int64_t ld, b200seq_step st, const b200seq_attn_desc a, float* __restrict__ kpool,
+                                      float* __restrict__ vpool, int* err) {
+    const int t = blockIdx.x;
+    const int Gv = a.vg > 0 ? a.vg : a.G;
+    const int nq = a.H * a.D, nk = a.G * a.D, nv = Gv * a.V;
+    int i = (blockIdx.y * blockDim.x + threadIdx.x) * VW;
+    if (i >= nq + nk + nv) return;
+    const bool isq = i < nq, isk = !isq && i < nq + nk;
+    i -= isq ? 0 : (isk ? nq : nq + nk);
+    const int col = (isq ? a.q_col : (isk ? a.k_col : a.v_col)) + i;
+    float* p = proj + (int64_t)t * ld + col;
+    float* dst = p;
+    if (!isq) {
+        const int64_t row = kv_row(st, st.tok_ent[t], st.tok_pos[t], err);
+        if (row < 0) return;
+        dst = isk ? kpool + row * nk + i : vpool + row * nv + i;
+    }
+    if (VW == 4) {
+        const float4 v = ld4(p), b = ld4(a.in_bias + col);
+        *reinterpret_cast<float4*>(dst) = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+    } else {
+        *dst = *p + a.in_bias[col];
+    }
+}
+
 // grid (T, column slices): the token that completes a block of P positions writes the block's mean key and mean value, one column per thread
 __global__ void attn_pool_kernel(b200seq_step st, int G, int D, int V, int P, int ppp, const float* __restrict__ kpool, const float* __restrict__ vpool,
                                  float* __restrict__ kpp, float* __restrict__ vpp, int* err) {
@@ -699,6 +726,17 @@ int b200seq_attn_prep_ex(float* proj, int64_t ld, const b200seq_step* st, const 
     if (st->T == 0) return 0;
     if (d->q_norm_w || d->k_norm_w || d->norm_full || d->rot_half || d->in_bias || d->kv_shared || d->vg > 0) {
         if (d->pool > 0 || d->v_col == d->k_col) return fail(B200SEQ_ERR_UNSUPPORTED, "attn_prep: the general form has no pooled blocks and own value columns");
+        if (d->in_bias && !d->q_norm_w && !d->k_norm_w && !d->norm_full && d->qk_eps < 0.f && d->rot_dims == 0 && !d->kv_shared) {
+            auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+            const bool vec = ((d->D | d->V | d->q_col | d->k_col | d->v_col) & 3) == 0 && (ld & 3) == 0 && al(proj) && al(d->in_bias) && al(kpool) && al(vpool);
+            const int cols = (d->H + d->G) * d->D + (d->vg > 0 ? d->vg : d->G) * d->V, nt = st->T <= 8 ? 64 : 256;
+            const int slices = ((vec ? cols / 4 : cols) + nt - 1) / nt;
+            if (slices > 65535) return fail(B200SEQ_ERR_UNSUPPORTED, "attn_prep: too many columns");
+            if (vec) attn_prep_bias_kernel<4><<<dim3(st->T, slices), nt, 0, (cudaStream_t)stream>>>(proj, ld, *st, *d, kpool, vpool, error_flag_dev());
+            else attn_prep_bias_kernel<1><<<dim3(st->T, slices), nt, 0, (cudaStream_t)stream>>>(proj, ld, *st, *d, kpool, vpool, error_flag_dev());
+            SEQ_LAUNCH_CHECK("attn_prep");
+            return 0;
+        }
         const int Dmax = d->D > d->V ? d->D : d->V;
         const size_t smem = (size_t)(d->rot_dims + 8 * Dmax + 40) * sizeof(float);
         if (smem > 48 * 1024) return fail(B200SEQ_ERR_UNSUPPORTED, "attn_prep: head size too large");

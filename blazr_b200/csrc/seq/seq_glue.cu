@@ -296,6 +296,37 @@ __global__ void causal_conv_kernel(const float* __restrict__ x, int64_t ldx, con
     }
 }
 
+// Steps in which every entry brings ONE token: grid (channel tiles, B), one channel per thread; state, taps and input are all requested before anything is
+// stored.  The same sums in the same order as above.
+__global__ void causal_conv_token_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ in_bias, const float* __restrict__ w,
+                                         const float* __restrict__ bias, float* __restrict__ state, b200seq_step st, int C, int taps, int mode, void* __restrict__ out,
+                                         int out_dtype, int64_t ldo, void* __restrict__ out2, int out2_dtype, int64_t ldo2) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, e = blockIdx.y;
+    if (c >= C) return;
+    const int t = st.ent_start[e], hist = taps - 1;
+    const bool fresh = st.ent_pos0[e] == 0;
+    float* sp = state + (int64_t)st.ent_slot[e] * hist * C + c;
+    float wr[MAX_TAPS], old[MAX_TAPS];
+#pragma unroll
+    for (int j = 0; j < MAX_TAPS; ++j) {
+        wr[j] = j < taps ? w[(int64_t)c * taps + j] : 0.f;
+        old[j] = (j < hist && !fresh) ? sp[(int64_t)j * C] : 0.f;
+    }
+    const float cur = x[(int64_t)t * ldx + c] + (in_bias ? in_bias[c] : 0.f), b = bias ? bias[c] : 0.f;
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < MAX_TAPS; ++j)
+        if (j < taps) acc = fmaf(wr[j], j == hist ? cur : old[j], acc);
+#pragma unroll
+    for (int j = 0; j < MAX_TAPS; ++j)
+        if (j < hist) sp[(int64_t)j * C] = j == hist - 1 ? cur : old[j + 1 < MAX_TAPS ? j + 1 : j];
+    float v = acc + b;
+    if (mode & B200SEQ_CONV_SILU) v = siluf_acc(v);
+    if (mode & B200SEQ_CONV_RESIDUAL) v = cur + v;
+    store_act(out, out_dtype, (int64_t)t * ldo + c, v);
+    if (out2) store_act(out2, out2_dtype, (int64_t)t * ldo2 + c, v);
+}
+
 // grid (T, groups): one block per norm group of a row
 __global__ void group_rmsnorm_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ w, int D, int groups, float eps,
                                      void* __restrict__ out, int out_dtype) {
@@ -338,9 +369,20 @@ __global__ void argmax_kernel(const float* __restrict__ logits, int V, int32_t* 
     const float* row = logits + (int64_t)blockIdx.x * V;
     float best = -INFINITY;
     int arg = 0x7fffffff;
-    for (int i = threadIdx.x; i < V; i += blockDim.x) {
-        const float v = row[i];
-        if (v > best || (v == best && i < arg)) best = v, arg = i;
+    if ((V & 3) == 0 && (reinterpret_cast<uintptr_t>(logits) & 15) == 0) {   // a thread's indices rise: the first of its equal values stays
+#pragma unroll 4
+        for (int i = threadIdx.x * 4; i < V; i += blockDim.x * 4) {
+            const float4 v = ld4(row + i);
+            if (v.x > best) best = v.x, arg = i;
+            if (v.y > best) best = v.y, arg = i + 1;
+            if (v.z > best) best = v.z, arg = i + 2;
+            if (v.w > best) best = v.w, arg = i + 3;
+        }
+    } else {
+        for (int i = threadIdx.x; i < V; i += blockDim.x) {
+            const float v = row[i];
+            if (v > best || (v == best && i < arg)) best = v, arg = i;
+        }
     }
     for (int o = 16; o > 0; o >>= 1) {
         const float ov = __shfl_xor_sync(0xffffffffu, best, o);
@@ -466,6 +508,13 @@ int b200seq_causal_conv_ex(const float* x, int64_t ldx, const float* in_bias, co
     if (out_dtype != B200SEQ_F32 && out_dtype != B200SEQ_BF16) return fail(B200SEQ_ERR_INVALID_ARG, "causal_conv: output dtype");
     if (out2 && ((out2_dtype != B200SEQ_F32 && out2_dtype != B200SEQ_BF16) || ldo2 < C)) return fail(B200SEQ_ERR_INVALID_ARG, "causal_conv: second output");
     if (st->T == 0) return 0;
+    if (st->T == st->B && st->B <= 65535) {
+        const int nt = C >= 4096 ? 128 : (C >= 1024 ? 64 : 32);
+        causal_conv_token_kernel<<<dim3((C + nt - 1) / nt, st->B), nt, 0, (cudaStream_t)stream>>>(x, ldx, in_bias, w, bias, state, *st, C, taps, mode, out, out_dtype, ldo, out2,
+                                                                                                 out2_dtype, ldo2);
+        SEQ_LAUNCH_CHECK("causal_conv");
+        return 0;
+    }
     const bool vec = C % 4 == 0 && ldx % 4 == 0 && ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
     if (vec) {
         dim3 grid((C / 4 + 127) / 128, (st->T + CONV_TILE - 1) / CONV_TILE);

@@ -7,6 +7,8 @@
 //             64 x 64 f32 fma tiles otherwise (exact 32-bit arithmetic; rows are gathered through the sort on load).
 //   combine : weighted sum of a token's expert outputs in choice order, plus an optional shared branch times a sigmoid token gate.
 // A pair's result depends on its token and expert only; which other tokens are in the step changes at most the kernel variant.
+#include <cooperative_groups.h>
+
 #include "seq_common.cuh"
 
 namespace b200seq {
@@ -163,16 +165,24 @@ __device__ __forceinline__ void bf16x8_f32(const uint4 v, float* f);
 template <typename XT>
 __device__ __forceinline__ float ldx(const XT* p);
 
-// Router of a step of few tokens in one kernel: grid (T), 8 warps.  The warps share out the NR rows of the router weight (the E experts'
-// rows and any rows stacked behind them), z[t][n] = x[t] . w[n] goes to memory and to shared memory, then warp 0 makes the token's choice.
+// Router of a step of few tokens in one kernel: a cluster of RT_CL blocks of 8 warps per token.  The cluster's warps share out the NR rows of the router
+// weight (the E experts' rows and any rows stacked behind them), z[t][n] = x[t] . w[n] goes to memory and to the first block's shared memory, whose
+// warp 0 then makes the token's choice.
+constexpr int RT_CL = 4;
 template <typename XT, bool VEC>
 __global__ void __launch_bounds__(256) moe_router_rows_kernel(const XT* __restrict__ x, int64_t ldx_, const __nv_bfloat16* __restrict__ w, int NR, int K,
                                                               float* __restrict__ z, int64_t ldz, const RouteRule rule, int32_t* __restrict__ ids,
                                                               float* __restrict__ wts) {
     extern __shared__ float sm[];   // NR logits, then the choice's 2 * E + groups floats
-    const int t = blockIdx.x, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+    namespace cg = cooperative_groups;
+    cg::cluster_group cl = cg::this_cluster();
+    const int cr = (int)cl.block_rank();
+    const int t = blockIdx.x / RT_CL, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
     const XT* xr = x + (int64_t)t * ldx_;
-    for (int n = wid; n < NR; n += 8) {
+    float* zs = cl.map_shared_rank(sm, 0);
+    auto here = cl.barrier_arrive();   // the first block runs before another one writes to its shared memory: waited for ahead of the first such write
+    bool waited = false;
+    for (int n = cr * 8 + wid; n < NR; n += 8 * RT_CL) {
         const __nv_bfloat16* wr = w + (int64_t)n * K;
         float acc = 0.f;
         if (VEC) {
@@ -193,13 +203,18 @@ __global__ void __launch_bounds__(256) moe_router_rows_kernel(const XT* __restri
             for (int k = lane; k < K; k += 32) acc = fmaf(__bfloat162float(wr[k]), ldx<XT>(xr + k), acc);
         }
         acc = warp_sum(acc);
+        if (!waited) {
+            cl.barrier_wait(std::move(here));
+            waited = true;
+        }
         if (lane == 0) {
-            sm[n] = acc;
+            zs[n] = acc;
             z[(int64_t)t * ldz + n] = acc;
         }
     }
-    __syncthreads();
-    if (wid == 0) route_token(sm, sm + NR, t, lane, rule, ids, wts, nullptr);
+    if (!waited) cl.barrier_wait(std::move(here));
+    cl.sync();
+    if (cr == 0 && wid == 0) route_token(sm, sm + NR, t, lane, rule, ids, wts, nullptr);
 }
 
 // grid (E), 256 threads: block e places the pairs of expert e behind those of the experts before it, in pair order
@@ -613,14 +628,22 @@ int b200seq_moe_router_rule(const void* x, int x_dtype, int64_t ldx_, const void
     const bool vec = K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (ldx_ * es) % 16 == 0;
     cudaStream_t cs = (cudaStream_t)stream;
     const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
-    if (x_dtype == B200SEQ_F32) {
-        if (vec) moe_router_rows_kernel<float, true><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
-        else moe_router_rows_kernel<float, false><<<T, 256, smem, cs>>>((const float*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
-    } else {
-        if (vec) moe_router_rows_kernel<__nv_bfloat16, true><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
-        else moe_router_rows_kernel<__nv_bfloat16, false><<<T, 256, smem, cs>>>((const __nv_bfloat16*)x, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
-    }
-    SEQ_LAUNCH_CHECK("moe_router");
+    cudaLaunchConfig_t cfg{};
+    cudaLaunchAttribute at{};
+    at.id = cudaLaunchAttributeClusterDimension;
+    at.val.clusterDim.x = RT_CL, at.val.clusterDim.y = 1, at.val.clusterDim.z = 1;
+    cfg.gridDim = dim3(T * RT_CL), cfg.blockDim = dim3(256), cfg.dynamicSmemBytes = smem, cfg.stream = cs, cfg.attrs = &at, cfg.numAttrs = 1;
+    const __nv_bfloat16* xb = (const __nv_bfloat16*)x;
+    const float* xf = (const float*)x;
+    cudaError_t e;
+    if (x_dtype == B200SEQ_F32)
+        e = vec ? cudaLaunchKernelEx(&cfg, moe_router_rows_kernel<float, true>, xf, ldx_, wb, NR, K, z, ldz, rule, ids, wts)
+                : cudaLaunchKernelEx(&cfg, moe_router_rows_kernel<float, false>, xf, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
+    else
+        e = vec ? cudaLaunchKernelEx(&cfg, moe_router_rows_kernel<__nv_bfloat16, true>, xb, ldx_, wb, NR, K, z, ldz, rule, ids, wts)
+                : cudaLaunchKernelEx(&cfg, moe_router_rows_kernel<__nv_bfloat16, false>, xb, ldx_, wb, NR, K, z, ldz, rule, ids, wts);
+    if (e != cudaSuccess) return cuda_status(e, "moe_router");
+    count_launch();
     return 0;
 }
 
